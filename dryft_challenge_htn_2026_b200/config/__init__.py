@@ -4,8 +4,9 @@ from .specs import (AttentionSpec, DenseMLPSpec, GatedLinearAttentionSpec, Gated
                     MaskedAttentionSpec, ModelSpec, OnePlusRMSNormSpec, ParallelMixerSpec, PostNormLayerSpec, RMSNormSpec,
                     RotaryHalfSpec, RotaryPairsSpec, RotaryPartSpec, RoutedMLPSpec, SandwichLayerSpec, ScalarRMSNormSpec, ScheduleEntry,
                     SinusoidSpec, UnitRMSNormSpec, LatentAttentionSpec, DiffAttentionSpec, GroupRMSNormSpec,
-                    LowerBoundRecurrenceSpec, StateSpaceSpec)
+                    LowerBoundRecurrenceSpec, StateSpaceSpec, BigramSpec, GatedDeltaSpec, LayerNormSpec, OutputNormLayerSpec)
 from .base import ConfigError, ModelConfig
+from .fukatar import FukatarConfig
 from .nevotar import NevotarConfig
 from .nilivik import NilivikConfig
 from .pibulix import PibulixConfig
@@ -17,4 +18,5 @@ __all__ = ["AttentionSpec", "DenseMLPSpec", "GatedMLPSpec", "LayerSpec", "Linear
            "SinusoidSpec", "ConfigError", "ModelConfig", "NilivikConfig", "Qwen3Config", "PibulixConfig",
            "GatedLinearAttentionSpec", "OnePlusRMSNormSpec", "PostNormLayerSpec", "RotaryPartSpec", "RoutedMLPSpec", "VenidraConfig", "LatentAttentionSpec", "RotaryPairsSpec",
            "SandwichLayerSpec", "UnitRMSNormSpec", "NevotarConfig", "DiffAttentionSpec", "GroupRMSNormSpec",
-           "LowerBoundRecurrenceSpec", "StateSpaceSpec"]
+           "LowerBoundRecurrenceSpec", "StateSpaceSpec", "FukatarConfig", "BigramSpec", "GatedDeltaSpec", "LayerNormSpec",
+           "OutputNormLayerSpec"]

@@ -52,6 +52,15 @@ class GroupRMSNormSpec:
 
 
 @dataclass(frozen=True)
+class LayerNormSpec:
+    """y = w * (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) over the last ``dim`` elements, no bias. ``tensor``: the
+    weight's name under the part's prefix (empty: the prefix itself names it)."""
+    dim: int
+    eps: float
+    tensor: str = ""
+
+
+@dataclass(frozen=True)
 class SinusoidSpec:
     """Absolute position vector added to the embedding: entry 2i = sin(p * base^(-2i/dim)), entry
     2i+1 = cos of the same angle."""
@@ -70,17 +79,23 @@ class RotaryHalfSpec:
 class RotaryPartSpec:
     """Rotate-half rotation of the first ``dim`` coordinates of a head (coordinate i with i + dim/2, i below
     dim/2) by angle(p, i) = p * base^(-2i/dim); the head's other coordinates pass. The frequencies are made in
-    float64 and rounded to float32 once; the angle is their float32 product with the position."""
+    float64 and rounded to float32 once; the angle is their float32 product with the position. ``scaling`` = (factor,
+    original, fast, slow) stretches the positions (YaRN): with at(t) = dim ln(original / (2 pi t)) / (2 ln base), lo =
+    max(floor(at(fast)), 0), hi = min(ceil(at(slow)), dim - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the
+    frequency of pair i is f_i (r_i / factor + 1 - r_i), and sine and cosine are multiplied by 0.1 ln(factor) + 1."""
     dim: int
     base: float
+    scaling: Optional[Tuple[float, float, float, float]] = None
 
 
 @dataclass(frozen=True)
 class RotaryPairsSpec:
     """Rotation of neighbouring pairs over the first ``dim`` coordinates of a vector (coordinate 2i with 2i + 1, i below
-    dim/2) by angle(p, i) = p * base^(-2i/dim); the other coordinates pass. Frequencies and angles as ``RotaryPartSpec``."""
+    dim/2) by angle(p, i) = p * base^(-2i/dim); the other coordinates pass. Frequencies, angles and ``scaling`` as
+    ``RotaryPartSpec``."""
     dim: int
     base: float
+    scaling: Optional[Tuple[float, float, float, float]] = None
 
 
 @dataclass(frozen=True)
@@ -120,7 +135,13 @@ class MaskedAttentionSpec:
     kernel and the split single-token kernel, which want a store of values, are not used then).
     ``bias``: q, k and v have biases (tensors ``q.b``, ``k.b``, ``v.b``), added in the projection. ``q_temp`` = (coef,
     every): q at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1). ``talk``: the heads' scores are
-    mixed before the masks and the softmax, score_h <- sum_g T[h, g] score_g with the tensor ``talk`` [heads, heads]."""
+    mixed before the masks and the softmax, score_h <- sum_g T[h, g] score_g with the tensor ``talk`` [heads, heads].
+    ``qk_norm_whole``: ``qk_norm`` (an ``RMSNormSpec`` or a ``UnitRMSNormSpec``) is taken of all rows of q, and of k, at
+    once before they are split into heads (tensors ``q.norm`` [heads * head_dim], ``k.norm`` [kv_heads * head_dim]), before
+    the rotation. ``position`` may also be a ``RotaryPairsSpec``. ``value_position`` (a rotation spec over v_head_dim): the
+    value of position j is turned by j and cached so, and each head's output at position i is turned back by i.
+    ``head_gate``: each head's output times the one number sigmoid(W_g x)_h (tensor ``g`` [heads, hidden]), after the
+    turning back."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -144,6 +165,9 @@ class MaskedAttentionSpec:
     bias: bool = False
     q_temp: Optional[Tuple[float, int]] = None
     talk: bool = False
+    qk_norm_whole: bool = False
+    value_position: Optional[Any] = None
+    head_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -198,6 +222,25 @@ class StateSpaceSpec:
 
 
 @dataclass(frozen=True)
+class GatedDeltaSpec:
+    """Gated delta rule. q = W_q x, k = W_k x (kv_heads x head_dim), v = W_v x (heads x v_head_dim), each through a causal
+    convolution per channel (``<q|k|v>.conv`` [channels, taps], last column the current token's) and SiLU; head h reads
+    q/k head h / (heads / kv_heads); q and k divided by sqrt(sum of squares + ``unit_eps``) per head, q times
+    head_dim^(-1/2); beta = sigmoid(W_b x), g = exp(-exp(A_log) softplus(W_a x + dt_bias)), one number a head. Per head S <-
+    g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q (state [head_dim, v_head_dim], float32, zero at the start). Each
+    head's o over its root mean square, times ``norm`` (shared by the heads), times silu(W_g x), then ``o``. The last taps -
+    1 inputs of the convolution are per-sequence state too."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    conv_taps: int
+    norm_eps: float
+    unit_eps: float = 1e-6
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Softmax attention whose queries, keys and values come through low-rank latents. With x the mixer's input:
     c_q = norm(W_dq x) (weight ``dq.norm``), q = W_uq c_q laid out head by head as [head_dim plain | rot_dim rotated];
@@ -217,6 +260,7 @@ class LatentAttentionSpec:
     position: Optional[Any] = None
     window: Optional[int] = None
     chunk: Optional[int] = None
+    sink: bool = False
 
 
 @dataclass(frozen=True)
@@ -253,15 +297,18 @@ class GatedLinearAttentionSpec:
 @dataclass(frozen=True)
 class ParallelMixerSpec:
     """Several mixers side by side on the same input; the result is the sum of scale_i * mixer_i(x).
-    ``branches``: (checkpoint prefix under the mixer, mixer spec, scale) each."""
+    ``branches``: (checkpoint prefix under the mixer, mixer spec, scale) each. ``out_norm_eps``: each branch's output goes
+    through an RMS norm over the width before the sum, with the weight ``<prefix>out`` and that eps inside the root."""
     hidden_size: int
     branches: Tuple[Tuple[str, Any, float], ...]
+    out_norm_eps: Optional[float] = None
 
 
 @dataclass(frozen=True)
 class DenseMLPSpec:
     """down(act(up(x))) without bias. ``activation`` "xielu": with two learned numbers p, q,
-    act(z) = softplus(p) z^2 + z/2 for z > 0 and (1/2 + softplus(q)) (e^z - 1 - z) + z/2 otherwise."""
+    act(z) = softplus(p) z^2 + z/2 for z > 0 and (1/2 + softplus(q)) (e^z - 1 - z) + z/2 otherwise; "relu2": act(z) =
+    max(z, 0)^2."""
     hidden_size: int
     intermediate_size: int
     activation: str = "xielu"
@@ -354,6 +401,34 @@ class SandwichLayerSpec:
 
 
 @dataclass(frozen=True)
+class OutputNormLayerSpec:
+    """One block with a norm on each sublayer's output alone: x <- x + norm_mix(mixer(x')), then x <- x + norm_ff(
+    feed_forward(x)). The sublayers read the stream itself; with ``shift`` (a tensor name under the prefix) the mixer reads
+    x' = x + (x_prev - x) * shift element by element, x_prev the stream of the token before at this place (zeros for the
+    first), which is per-sequence state; without it x' = x. Without a feed-forward the second step, its norm and their
+    names fall away."""
+    prefix: str
+    mixer: Any
+    norm_mix: Any
+    feed_forward: Any
+    norm_ff: Any
+    shift: Optional[str] = None
+    names: Tuple[Tuple[str, str], ...] = (("mixer", "mix."), ("norm_mix", "norm1"), ("feed_forward", "mlp."),
+                                          ("norm_ff", "norm2"))
+
+
+@dataclass(frozen=True)
+class BigramSpec:
+    """Rows of a table of token pairs that the embedding adds: row (previous * mul_prev + token * mul_cur) mod buckets, and
+    row ``buckets`` (the last) for a sequence's first token. ``tensor`` [buckets + 1, hidden]. The previous token is
+    per-sequence state of the model."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+    tensor: str = "bigram"
+
+
+@dataclass(frozen=True)
 class ScheduleEntry:
     """One run of a layer. ``cache`` names the cache entry the layer's mixer uses; with
     ``writes=False`` the mixer only reads what the entry's owner stored in this step. Right before the
@@ -384,6 +459,7 @@ class ModelSpec:
     logit_cap: Optional[float] = None          # logits <- cap * tanh(logits / cap)
     logit_scale: float = 1.0                   # multiplies the logits before the cap
     tables: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()   # learned float32 tables of the model itself: (checkpoint name, shape)
+    embed_bigram: Optional[BigramSpec] = None  # rows of token pairs added to the (scaled) embedding
     unused_tensors: Tuple[str, ...] = ()       # checkpoint names the design ships although nothing reads them
     extra: dict = field(default_factory=dict, compare=False)
 

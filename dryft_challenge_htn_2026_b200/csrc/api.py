@@ -306,6 +306,7 @@ def attention_decode_bf16(q, out, k_store, v_store, row_pos, page_table, n_heads
 
 # ---------------------------------------------------------------------------------------- products
 MODE_STORE, MODE_STORE_F32, MODE_SILU, MODE_XIELU = 0, 1, 2, 3
+RELU2 = (1.0, -1.0)         # ``act`` of a MODE_XIELU product: the squared ReLU (a negative second constant selects it)
 GATE_GELU = (1.0, 0.0)      # ``act`` of a MODE_SILU product whose gate goes through the tanh form of GELU instead of SiLU
 
 
@@ -664,7 +665,7 @@ def softcap(x, cap, factor=1.0):
 
 
 def xielu(z, out, alpha_pos, alpha_neg):
-    """out = alpha_pos z^2 + z/2 (z > 0), alpha_neg (e^z - 1 - z) + z/2 (z <= 0)."""
+    """out = alpha_pos z^2 + z/2 (z > 0), alpha_neg (e^z - 1 - z) + z/2 (z <= 0); ``RELU2`` as the constants: max(z, 0)^2."""
     _need(z, "z", None), _need(out, "out", z.dtype)
     if out.shape != z.shape:
         raise KernelError("xielu: shapes do not match")
@@ -732,7 +733,8 @@ def masked_bf16_takes(head_dim, v_head_dim):
 
 
 def attention_masked_prefill_bf16(q, out, gate, out_scale, k_store, v_store, tiles, cu_q, seq_pos0, page_table, n_heads,
-                                  n_kv_heads, head_dim, v_head_dim, window, chunk, scale, r1=None, r2=None, sink=None):
+                                  n_kv_heads, head_dim, v_head_dim, window, chunk, scale, r1=None, r2=None, sink=None,
+                                  softcap=None):
     """``attention_masked`` for ragged query portions on the tensor cores (bfloat16). tiles [n, 2] int32 =
     (sequence, first query of a 64-row tile within its portion); cu_q [nseq+1]; seq_pos0 [nseq]."""
     _need_rows(q, "q", torch.bfloat16), _need_rows(out, "out", torch.bfloat16), _need_rows(gate, "gate", torch.bfloat16)
@@ -747,7 +749,7 @@ def attention_masked_prefill_bf16(q, out, gate, out_scale, k_store, v_store, til
                                                 c_longlong(gate.stride(0) if gate is not None else 0), c_float(out_scale),
                                                 _p(k_store), _p(v_store), _p(tiles), tiles.shape[0], _p(cu_q), _p(seq_pos0),
                                                 _p(page_table), page_table.shape[1], n_heads, n_kv_heads, int(window or 0),
-                                                int(chunk or 0), c_float(scale), _p(r1), _p(r2), _p(sink), _stream()),
+                                                int(chunk or 0), c_float(scale), c_float(softcap or 0.0), _p(r1), _p(r2), _p(sink), _stream()),
            "attention_masked_prefill_bf16")
 
 
@@ -781,12 +783,13 @@ def shared_rows_ws(rows, n_heads, v_head_dim, nsplit, device):
 
 
 def attention_shared_rows_bf16(q, out, out_scale, k_store, page_table, n_heads, n_kv_heads, head_dim, v_head_dim, window, chunk,
-                               scale, tiles=None, cu_q=None, seq_pos0=None, row_pos=None, nsplit=1, ws=None):
+                               scale, tiles=None, cu_q=None, seq_pos0=None, row_pos=None, nsplit=1, ws=None, sink=None):
     """Masked softmax attention (bfloat16, mma.sync) whose values are the first ``v_head_dim`` numbers of the cached key
     rows, all query heads of a group in one block. Prompts: ``tiles`` [n, 2] = (sequence, first query of a tile of
     ``shared_rows_tile_queries`` queries), ``cu_q``, ``seq_pos0``. Single tokens: ``row_pos`` [rows] (negative: padding),
-    page table row i for row i, the keys of a row in ``nsplit`` runs with ``ws`` = ``shared_rows_ws`` when nsplit > 1."""
-    _need_rows(q, "q", torch.bfloat16), _need_rows(out, "out", torch.bfloat16)
+    page table row i for row i, the keys of a row in ``nsplit`` runs with ``ws`` = ``shared_rows_ws`` when nsplit > 1.
+    ``sink`` (float32 [n_heads]): its exponential joins the denominator."""
+    _need_rows(q, "q", torch.bfloat16), _need_rows(out, "out", torch.bfloat16), _need(sink, "sink", torch.float32, 1)
     _need(page_table, "page_table", torch.int32, 2), _need(k_store, "k_store", torch.bfloat16)
     if not shared_rows_takes(head_dim, v_head_dim) or n_heads % n_kv_heads or not shared_rows_operands(q, out):
         raise KernelError(f"attention_shared_rows_bf16: sizes {head_dim}/{v_head_dim}, head counts or row strides not supported")
@@ -802,7 +805,7 @@ def attention_shared_rows_bf16(q, out, out_scale, k_store, page_table, n_heads, 
     _check(lib, lib.dk_attn_shared_rows_bf16(_p(q), c_longlong(q.stride(0)), _p(out), c_longlong(out.stride(0)), c_float(out_scale),
                                              _p(k_store), _p(tiles), n_items, _p(cu_q), _p(seq_pos0), _p(row_pos), _p(page_table),
                                              page_table.shape[1], n_heads, n_kv_heads, int(window or 0), int(chunk or 0),
-                                             c_float(scale), nsplit, _p(ws[0]) if nsplit > 1 else None,
+                                             c_float(scale), _p(sink), nsplit, _p(ws[0]) if nsplit > 1 else None,
                                              _p(ws[1]) if nsplit > 1 else None, _stream()),
            "attention_shared_rows_bf16", kernels=2 if nsplit > 1 else 1)
 
@@ -918,7 +921,7 @@ def masked_decode_ws(rows, n_heads, v_head_dim, nsplit, device):
 
 def attention_masked_decode_bf16(q, out, gate, out_scale, k_store, v_store, row_pos, page_table, n_heads, n_kv_heads,
                                  head_dim, v_head_dim, window, chunk, scale, span, r1=None, r2=None, sink=None,
-                                 k_new=None, v_new=None, ws=None):
+                                 k_new=None, v_new=None, ws=None, softcap=None):
     """``attention_masked`` for one query token per sequence (bfloat16 storage, float32 arithmetic): a block
     per (kv head, row, run of keys) for all query heads of the group, and a merge kernel when the keys are
     split. ``span`` = (keys a block, splits) from ``masked_decode_span``, ``ws`` from ``masked_decode_ws``. With
@@ -943,7 +946,7 @@ def attention_masked_decode_bf16(q, out, gate, out_scale, k_store, v_store, row_
                                                c_longlong(gate.stride(0) if gate is not None else 0), c_float(out_scale),
                                                _p(k_store), _p(v_store), _p(row_pos), _p(page_table), page_table.shape[1],
                                                q.shape[0], n_heads, n_kv_heads, int(window or 0), int(chunk or 0),
-                                               c_float(scale), _p(r1), _p(r2), _p(sink), int(span), _p(k_new), _p(v_new),
+                                               c_float(scale), c_float(softcap or 0.0), _p(r1), _p(r2), _p(sink), int(span), _p(k_new), _p(v_new),
                                                c_longlong(k_new.stride(0) if k_new is not None else 0), nsplit,
                                                _p(ws[0] if nsplit > 1 else None), _p(ws[1] if nsplit > 1 else None), _stream()),
            "attention_masked_decode_bf16", 1 if nsplit == 1 else 2)
@@ -1178,12 +1181,13 @@ def latent_norm_rope_write(proj, cq_out, q_norm_w, kv_norm_w, eps, cos, sin, rot
     rmsnorm(b) * kv_norm_w and r, its first ``rot_dims`` coordinates rotated by neighbouring pairs (cos/sin
     [positions, rot_dims/2]), go to each token's place in the paged cache of one kv head: key row [c | r]
     (k_store [pages, 1, PAGE, kv_rank + rot_dim]), and, where the cache keeps a store of values, value row c
-    (v_store [pages, 1, PAGE, kv_rank] or None)."""
+    (v_store [pages, 1, PAGE, kv_rank] or None). ``q_rank`` 0: rows [b | r], ``cq_out`` and ``q_norm_w`` None."""
     _need_rows(proj, "proj"), _need_rows(cq_out, "cq_out", proj.dtype)
     _need(q_norm_w, "q_norm_w", torch.float32, 1), _need(kv_norm_w, "kv_norm_w", torch.float32, 1)
     _need(cos, "cos", torch.float32, 2), _need(sin, "sin", torch.float32, 2)
     _need(row_pos, "row_pos", torch.int32, 1), _need(row_seq, "row_seq", torch.int32, 1)
-    if proj.shape[1] != q_rank + kv_rank + rot_dim or cq_out.shape != (proj.shape[0], q_rank) or q_norm_w.numel() != q_rank \
+    if proj.shape[1] != q_rank + kv_rank + rot_dim or (q_rank > 0 and (cq_out is None or cq_out.shape != (proj.shape[0], q_rank)
+                                                                       or q_norm_w is None or q_norm_w.numel() != q_rank)) \
             or kv_norm_w.numel() != kv_rank or rot_dims % 2 or rot_dims > rot_dim or \
             (rot_dims and (cos is None or cos.shape[1] != rot_dims // 2 or sin.shape != cos.shape)):
         raise KernelError("latent_norm_rope_write: shapes do not match")
@@ -1192,8 +1196,8 @@ def latent_norm_rope_write(proj, cq_out, q_norm_w, kv_norm_w, eps, cos, sin, rot
         if k_store.shape[1:] != (1, PAGE, kv_rank + rot_dim) or (v_store is not None and v_store.shape[1:] != (1, PAGE, kv_rank)):
             raise KernelError("latent_norm_rope_write: key/value stores of the wrong shape")
     lib = _lib("latent.cu")
-    _check(lib, lib.dk_latent_norm_rope_write(_dt(proj), _p(proj), c_longlong(proj.stride(0)), _p(cq_out), c_longlong(cq_out.stride(0)),
-                                              _p(q_norm_w), _p(kv_norm_w), c_float(eps), _p(cos), _p(sin), int(rot_dims),
+    _check(lib, lib.dk_latent_norm_rope_write(_dt(proj), _p(proj), c_longlong(proj.stride(0)), _p(cq_out),
+                                              c_longlong(cq_out.stride(0) if cq_out is not None else 0), _p(q_norm_w), _p(kv_norm_w), c_float(eps), _p(cos), _p(sin), int(rot_dims),
                                               _p(row_pos), _p(row_seq), proj.shape[0], q_rank, kv_rank, rot_dim, _p(k_store),
                                               _p(v_store), _p(page_table), page_table.shape[1] if page_table is not None else 0,
                                               _stream()), "latent_norm_rope_write")
@@ -1581,3 +1585,227 @@ def attention_talk_bf16(q, out, out_scale, k_store, v_store, page_table, n_heads
                                            _p(talk), int(nsplit), _p(ws[0]) if ws is not None else c_void_p(0),
                                            _p(ws[1]) if ws is not None else c_void_p(0), _stream()),
            "attention_talk_bf16", 2 if nsplit > 1 else 1)
+
+
+# ------------------------------------------- the stream of blocks that norm a sublayer's output, and the shift between tokens
+class NormedSum:
+    """A sublayer's output as factor * sum_i rms(d_i) * w_i of one or two products' outputs (tensors or ``Partial``), each
+    over its own root mean square over the width (eps inside the root): worked out by the kernel that adds it to the stream."""
+
+    def __init__(self, deltas, weights, eps, factor):
+        if not 1 <= len(deltas) <= 2 or len(weights) != len(deltas):
+            raise ValueError("one or two outputs, each with its weight")
+        self.deltas, self.weights, self.eps, self.factor = list(deltas), list(weights), float(eps), float(factor)
+
+    def to_float32(self):
+        out = 0.0
+        for d, w in zip(self.deltas, self.weights):
+            d = d.ws.sum(0) if isinstance(d, Partial) else d.to(torch.float32)
+            out = out + d * torch.rsqrt((d * d).mean(-1, keepdim=True) + self.eps) * w
+        return self.factor * out
+
+
+def _add_args(h, delta, norm, dtype, what):
+    """The C arguments of what joins the stream: sources, their norms, the norm of their sum. ``norm``: None or (weight, eps,
+    center)."""
+    normed = isinstance(delta, NormedSum)
+    sources = delta.deltas if normed else [] if delta is None else [delta]
+    args = []
+    for i in range(2):
+        src = sources[i] if i < len(sources) else None
+        x, parts, n, stride = _parts(src)
+        _need(x, "delta", dtype, 2)
+        w = delta.weights[i] if normed and src is not None else None
+        _need(w, "delta weight", torch.float32, 1)
+        if (src is not None and tuple(src.shape) != tuple(h.shape)) or (w is not None and w.numel() != h.shape[1]):
+            raise KernelError(f"{what}: shapes do not match")
+        args += [_p(x), parts, n, stride if src is not None else c_longlong(0), _p(w)]
+    nw, eps, center = norm if norm is not None else (None, 0.0, False)
+    _need(nw, "norm weight", torch.float32, 1)
+    if nw is not None and nw.numel() != h.shape[1]:
+        raise KernelError(f"{what}: shapes do not match")
+    return args + [c_float(delta.eps if normed else 0.0), c_float(delta.factor if normed else 1.0), _p(nw), c_float(eps),
+                   int(bool(center))]
+
+
+def _need_sequences(row_pos, row_seq, cu_q, seq_slot, rows):
+    for t, n in ((row_pos, "row_pos"), (row_seq, "row_seq"), (cu_q, "cu_q"), (seq_slot, "seq_slot")):
+        _need(t, n, torch.int32, 1)
+    if row_pos.numel() < rows or row_seq.numel() < rows:
+        raise KernelError("positions and sequences of every row are needed")
+
+
+def sublayer_add(h, delta, norm, a_out, h_out=None, rows=None, next_norm=None, save=None, seqs=None):
+    """h_out = h + norm(delta) (float32), a_out = that row in its own type, or ``next_norm`` of it. ``delta``: None, a tensor,
+    a ``Partial`` or a ``NormedSum``; ``norm`` and ``next_norm``: None or (weight, eps, center), center True for a layer norm.
+    ``rows`` (int32): a_out row i is made of h row rows[i], h_out is not written. ``save`` (float32 [slots, H]): h as it stood
+    before the sum goes there at every sequence's last row, ``seqs`` = (row_pos, row_seq, cu_q or None, seq_slot)."""
+    _need(h, "h", torch.float32, 2), _need(h_out, "h_out", torch.float32, 2), _need(a_out, "a_out", None, 2)
+    _need(rows, "rows", torch.int32, 1), _need(save, "save", torch.float32, 2)
+    n = h.shape[0] if rows is None else rows.numel()
+    if tuple(a_out.shape) != (n, h.shape[1]) or (h_out is not None and (h_out.shape != h.shape or rows is not None)) \
+            or (save is not None and (seqs is None or save.shape[1] != h.shape[1] or rows is not None)):
+        raise KernelError("sublayer_add: shapes do not match")
+    args = _add_args(h, delta, norm, a_out.dtype, "sublayer_add")
+    nw, neps, ncenter = next_norm if next_norm is not None else (None, 0.0, False)
+    _need(nw, "next norm weight", torch.float32, 1)
+    row_pos, row_seq, cu_q, seq_slot = seqs if seqs is not None else (None,) * 4
+    if save is not None:
+        _need_sequences(row_pos, row_seq, cu_q, seq_slot, h.shape[0])
+    lib = _lib("stream.cu")
+    _check(lib, lib.dk_sublayer_add(_dt(a_out), _p(h), _p(h_out), *args, _p(rows), _p(nw), c_float(neps), int(bool(ncenter)),
+                                    _p(a_out), _p(save), _p(row_pos), _p(row_seq), _p(cu_q), _p(seq_slot), n, h.shape[1],
+                                    _stream()), "sublayer_add")
+
+
+def sublayer_add_shift(h, delta, norm, share, state, seqs, a_out, h_out=None):
+    """x = h + norm(delta) -> h_out (another buffer than h; not needed without a delta), a_out = x + (x_prev - x) * share with
+    x_prev the row of the token before: the row above, or ``state`` [slots, H] at the first row a sequence brings.
+    ``seqs`` = (row_pos, row_seq, cu_q or None, seq_slot); ``cu_q`` None: one token a row."""
+    _need(h, "h", torch.float32, 2), _need(h_out, "h_out", torch.float32, 2), _need(a_out, "a_out", None, 2)
+    _need(share, "share", torch.float32, 1), _need(state, "state", torch.float32, 2)
+    row_pos, row_seq, cu_q, seq_slot = seqs
+    n, H = h.shape
+    _need_sequences(row_pos, row_seq, cu_q, seq_slot, n)
+    if a_out.shape != h.shape or share.numel() != H or state.shape[1] != H or (h_out is None) != (delta is None) or \
+            (h_out is not None and (h_out.shape != h.shape or h_out.data_ptr() == h.data_ptr())):
+        raise KernelError("sublayer_add_shift: shapes do not match, or h_out is h")
+    args = _add_args(h, delta, norm, a_out.dtype, "sublayer_add_shift")
+    run = 1 if cu_q is None or n < 4 * sm_count() else 4        # rows a block: the row ahead of them is worked out twice
+    lib = _lib("stream.cu")
+    _check(lib, lib.dk_sublayer_add_shift(_dt(a_out), _p(h), _p(h_out), *args, _p(share), _p(state), _p(row_pos), _p(row_seq), _p(cu_q),
+                                          _p(seq_slot), n, run, _p(a_out), H, _stream()), "sublayer_add_shift")
+
+
+def stream_save(h, state, cu_q, seq_pos0, seq_slot, n_seq):
+    """state[slot] <- h at every sequence's last row (``cu_q`` None: row s is sequence s; seq_pos0[s] < 0: padding)."""
+    _need(h, "h", torch.float32, 2), _need(state, "state", torch.float32, 2), _need(cu_q, "cu_q", torch.int32, 1)
+    _need(seq_pos0, "seq_pos0", torch.int32, 1), _need(seq_slot, "seq_slot", torch.int32, 1)
+    if state.shape[1] != h.shape[1]:
+        raise KernelError("stream_save: shapes do not match")
+    lib = _lib("stream.cu")
+    _check(lib, lib.dk_stream_save(_p(h), _p(state), _p(cu_q), _p(seq_pos0), _p(seq_slot), n_seq, h.shape[1], _stream()), "stream_save")
+
+
+def embed_bigram(tok, embed, scale, table, mul_prev, mul_cur, state, seqs, h_out):
+    """h_out[t] = embed[tok[t]] * scale + table[row], row = (previous token * mul_prev + tok[t] * mul_cur) mod buckets with
+    buckets + 1 rows in the table, the last of them for position 0. ``state`` int32 [slots, 1]: the last token of every
+    sequence, read for the first row it brings and moved on. ``seqs`` as in ``sublayer_add_shift``."""
+    _need(tok, "tok", torch.int32, 1), _need(embed, "embed", None, 2), _need(table, "table", embed.dtype, 2)
+    _need(state, "state", torch.int32, 2), _need(h_out, "h_out", torch.float32, 2)
+    row_pos, row_seq, cu_q, seq_slot = seqs
+    n, (V, H) = tok.numel(), embed.shape
+    _need_sequences(row_pos, row_seq, cu_q, seq_slot, n)
+    if table.shape[1] != H or table.shape[0] < 2 or tuple(h_out.shape) != (n, H) or state.shape[1] != 1 or mul_prev < 0 or mul_cur < 0:
+        raise KernelError("embed_bigram: shapes do not match, or a negative multiplier")
+    lib = _lib("stream.cu")
+    _check(lib, lib.dk_embed_bigram(_dt(embed), _p(tok), _p(embed), c_float(scale), _p(table), table.shape[0] - 1, c_longlong(mul_prev),
+                                    c_longlong(mul_cur), _p(state), _p(row_pos), _p(row_seq), _p(cu_q), _p(seq_slot), n, H, V,
+                                    _p(h_out), _stream()), "embed_bigram")
+
+
+# --------------------------------------------------- between an attention mixer's projection and its cache, and behind it
+NORM_WHOLE = 3
+
+
+def qkv_rows(proj, q_out, norm_mode, q_norm_w, k_norm_w, eps, rot, v_rot, row_pos, row_seq, n_heads, n_kv_heads, head_dim, v_head_dim,
+             k_store=None, v_store=None, page_table=None):
+    """Rows [q | k | v] of a projection -> ``q_out`` [tokens, heads * head_dim] and, with the paged stores, each token's k and
+    v heads at their place there. ``norm_mode``: NORM_NONE, NORM_BEFORE_ROTATION, NORM_AFTER_ROTATION (per head, weights of
+    the head's size or None) or NORM_WHOLE (all heads at once before the rotation, weights of the whole projection's size or
+    None). ``rot`` and ``v_rot``: None or (cos, sin [positions, dims / 2], dims, pairs): the rotation of the first ``dims``
+    coordinates of q and k heads, and that of whole value heads."""
+    _need_rows(proj, "proj"), _need_rows(q_out, "q_out", proj.dtype)
+    _need(q_norm_w, "q_norm_w", torch.float32, 1), _need(k_norm_w, "k_norm_w", torch.float32, 1)
+    _need(row_pos, "row_pos", torch.int32, 1), _need(row_seq, "row_seq", torch.int32, 1)
+    n_q, n_k = n_heads * head_dim, n_kv_heads * head_dim
+    for r, nm, limit in ((rot, "rot", head_dim), (v_rot, "v_rot", v_head_dim)):
+        if r is not None:
+            _need(r[0], nm, torch.float32, 2), _need(r[1], nm, torch.float32, 2)
+            if r[2] % 2 or r[2] > limit or r[0].shape[1] != r[2] // 2 or r[1].shape != r[0].shape:
+                raise KernelError(f"qkv_rows: {nm} over {r[2]} coordinates of {limit}")
+    sizes = (n_q, n_k) if norm_mode == NORM_WHOLE else (head_dim, head_dim)
+    if proj.shape[1] != n_q + n_k + n_kv_heads * v_head_dim or q_out.shape != (proj.shape[0], n_q) or max(head_dim, v_head_dim) > 256 \
+            or any(w is not None and w.numel() != n for w, n in zip((q_norm_w, k_norm_w), sizes)) \
+            or (v_rot is not None and v_rot[2] != v_head_dim):
+        raise KernelError("qkv_rows: shapes do not match")
+    if k_store is not None:
+        _need(k_store, "k_store", proj.dtype, 4), _need(v_store, "v_store", proj.dtype, 4), _need(page_table, "page_table", torch.int32, 2)
+        if k_store.shape[1:] != (n_kv_heads, PAGE, head_dim) or v_store is None or v_store.shape[1:] != (n_kv_heads, PAGE, v_head_dim):
+            raise KernelError("qkv_rows: key/value stores of the wrong shape")
+    cos, sin, dims, pairs = rot if rot is not None else (None, None, 0, False)
+    vcos, vsin, _, v_pairs = v_rot if v_rot is not None else (None, None, 0, False)
+    lib = _lib("qkv_rows.cu")
+    _check(lib, lib.dk_qkv_rows(_dt(proj), _p(proj), c_longlong(proj.stride(0)), _p(q_out), c_longlong(q_out.stride(0)), int(norm_mode),
+                                _p(q_norm_w), _p(k_norm_w), c_float(eps), _p(cos), _p(sin), int(dims), int(bool(pairs)), _p(vcos),
+                                _p(vsin), int(bool(v_pairs)), _p(row_pos), _p(row_seq), proj.shape[0], n_heads, n_kv_heads, head_dim,
+                                v_head_dim, _p(k_store), _p(v_store), _p(page_table),
+                                page_table.shape[1] if page_table is not None else 0, _stream()), "qkv_rows")
+
+
+def turn_back_gate(o, out, gate, v_rot, out_scale, row_pos, n_heads, v_head_dim):
+    """out = per head ``o`` turned back by the row's position (``v_rot`` as in ``qkv_rows``, or None) * sigmoid(gate[t, h]) *
+    out_scale; ``gate`` [tokens, heads] or None. o, out and gate may be rows of wider matrices."""
+    _need_rows(o, "o"), _need_rows(out, "out", o.dtype), _need_rows(gate, "gate", o.dtype), _need(row_pos, "row_pos", torch.int32, 1)
+    if o.shape[1] != n_heads * v_head_dim or out.shape != o.shape or v_head_dim % 2 or (gate is not None and gate.shape != (o.shape[0], n_heads)) \
+            or (v_rot is not None and (v_rot[2] != v_head_dim or v_rot[0].shape[1] != v_head_dim // 2)):
+        raise KernelError("turn_back_gate: shapes do not match (value heads of even size)")
+    cos, sin, _, pairs = v_rot if v_rot is not None else (None, None, 0, False)
+    lib = _lib("qkv_rows.cu")
+    _check(lib, lib.dk_turn_back_gate(_dt(o), _p(o), c_longlong(o.stride(0)), _p(out), c_longlong(out.stride(0)), _p(gate),
+                                      c_longlong(gate.stride(0) if gate is not None else 0), _p(cos), _p(sin), int(bool(pairs)),
+                                      c_float(out_scale), _p(row_pos), o.shape[0], n_heads, v_head_dim, _stream()), "turn_back_gate")
+
+
+# ------------------------------------------------------------------------------------------------ gated delta rule
+def delta_operands(rows, n_heads, n_kv_heads, head_dim, v_head_dim, device):
+    """(qkv, scal): float32 [rows, 2 * n_kv_heads * head_dim + n_heads * v_head_dim] unit queries and keys and the values, and
+    float32 [rows, 2 * n_heads + n_kv_heads] decays, step sizes and k . q."""
+    return (torch.empty((rows, 2 * n_kv_heads * head_dim + n_heads * v_head_dim), dtype=torch.float32, device=device),
+            torch.empty((rows, 2 * n_heads + n_kv_heads), dtype=torch.float32, device=device))
+
+
+def delta_prepare(proj, a_rows, b_rows, state, w_conv, taps, a_log, dt_bias, unit_eps, row_pos, row_seq, seq_pos0, seq_slot, qkv, scal,
+                  n_heads, n_kv_heads, head_dim, v_head_dim):
+    """proj rows [q | k | v] -> the recurrence's operands (``delta_operands``): causal convolution per channel with ``w_conv``
+    [channels, taps] (``state`` [slots, taps - 1, channels] for positions before the step, read only: ``conv_state_update``
+    moves it on), SiLU, unit queries (times head_dim^(-1/2)) and keys; decays exp(-exp(a_log) softplus(a + dt_bias)), step
+    sizes sigmoid(b). ``a_rows``, ``b_rows`` [T, heads]: columns of the matrix that holds ``proj``."""
+    _need_rows(proj, "proj"), _need_rows(a_rows, "a_rows", proj.dtype), _need_rows(b_rows, "b_rows", proj.dtype)
+    _need(state, "state", proj.dtype, 3), _need(w_conv, "w_conv", proj.dtype, 2)
+    _need(a_log, "a_log", torch.float32, 1), _need(dt_bias, "dt_bias", torch.float32, 1)
+    _need(qkv, "qkv", torch.float32, 2), _need(scal, "scal", torch.float32, 2)
+    for t, nm in ((row_pos, "row_pos"), (row_seq, "row_seq"), (seq_pos0, "seq_pos0"), (seq_slot, "seq_slot")):
+        _need(t, nm, torch.int32, 1)
+    T, C = proj.shape
+    if C != 2 * n_kv_heads * head_dim + n_heads * v_head_dim or qkv.shape != (T, C) or scal.shape != (T, 2 * n_heads + n_kv_heads) \
+            or tuple(w_conv.shape) != (C, taps) or a_rows.shape != (T, n_heads) or b_rows.shape != (T, n_heads) \
+            or not (a_rows.stride(0) == b_rows.stride(0) == proj.stride(0)) or n_heads % n_kv_heads \
+            or a_log.numel() != n_heads or dt_bias.numel() != n_heads or not 1 <= taps <= SHORT_CONV_MAX_TAPS \
+            or (taps > 1 and (state is None or tuple(state.shape[1:]) != (taps - 1, C))):
+        raise KernelError("delta_prepare: shapes do not match")
+    lib = _lib("delta_rule.cu")
+    _check(lib, lib.dk_delta_prepare(_dt(proj), _p(proj), c_longlong(proj.stride(0)), _p(a_rows), _p(b_rows), _p(state), _p(w_conv),
+                                     int(taps), _p(a_log), _p(dt_bias), c_float(unit_eps), _p(row_pos), _p(row_seq), _p(seq_pos0),
+                                     _p(seq_slot), _p(qkv), _p(scal), T, n_heads, n_kv_heads, head_dim, v_head_dim, _stream()),
+           "delta_prepare")
+
+
+def delta_rule(qkv, scal, out, state, cu_q, seq_pos0, seq_slot, n_seq, n_heads, n_kv_heads, head_dim, v_head_dim):
+    """S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q per (sequence, head), token by token, all float32, over the
+    operands of ``delta_prepare``; state [slots, n_heads, head_dim, v_head_dim], out [T, n_heads * v_head_dim]. Rows of
+    sequence s are cu_q[s] .. cu_q[s + 1]; ``cu_q`` None: row s alone (its position seq_pos0[s] < 0: padding)."""
+    _need(qkv, "qkv", torch.float32, 2), _need(scal, "scal", torch.float32, 2), _need(out, "out", torch.float32, 2)
+    _need(state, "state", torch.float32, 4), _need(cu_q, "cu_q", torch.int32, 1)
+    _need(seq_pos0, "seq_pos0", torch.int32, 1), _need(seq_slot, "seq_slot", torch.int32, 1)
+    T = qkv.shape[0]
+    if qkv.shape[1] != 2 * n_kv_heads * head_dim + n_heads * v_head_dim or scal.shape != (T, 2 * n_heads + n_kv_heads) \
+            or out.shape != (T, n_heads * v_head_dim) or tuple(state.shape[1:]) != (n_heads, head_dim, v_head_dim) or head_dim > 256:
+        raise KernelError("delta_rule: shapes do not match (key sizes up to 256)")
+    lib = _lib("delta_rule.cu")
+    if cu_q is None:
+        _check(lib, lib.dk_delta_rule_step(_p(qkv), _p(scal), _p(out), _p(state), _p(seq_pos0), _p(seq_slot), T, n_heads, n_kv_heads,
+                                           head_dim, v_head_dim, _stream()), "delta_rule")
+    else:
+        _check(lib, lib.dk_delta_rule(_p(qkv), _p(scal), _p(out), _p(state), _p(cu_q), _p(seq_pos0), _p(seq_slot), n_seq, n_heads,
+                                      n_kv_heads, head_dim, v_head_dim, _stream()), "delta_rule")

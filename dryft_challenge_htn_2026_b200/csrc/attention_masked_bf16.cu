@@ -42,11 +42,16 @@ __device__ __forceinline__ void stage_page_kv(bf16* stage, const bf16* k_store, 
     }
 }
 
+// tanh(y) from one exponential and one division
+__device__ __forceinline__ float capped_unit(float y) { return 1.f - __fdividef(2.f, __expf(2.f * y) + 1.f); }
+
 // One warp: 16 query rows against the 64 staged keys of a page. Row r (0: lane group g, 1: g+8) sits at
-// position hi[r] and may see keys lo[r] <= position <= hi[r]. Scores in the log2 domain.
+// position hi[r] and may see keys lo[r] <= position <= hi[r]. Scores in the log2 domain. cap2 = cap * log2(e) and cap_in
+// = scale / cap where the scores are capped (score = cap * tanh(score / cap)), cap2 = 0 where not.
 __device__ __forceinline__ void warp_attend_masked(const uint32_t (&qf)[HD / 16][4], const bf16* Ks, const bf16* Vs,
-                                                   int key0, const int (&lo)[2], const int (&hi)[2], float sl2, float b1,
-                                                   float b2, float (&m)[2], float (&l)[2], float (&acc)[HDV / 8][4]) {
+                                                   int key0, const int (&lo)[2], const int (&hi)[2], float sl2, float cap2,
+                                                   float cap_in, float b1, float b2, float (&m)[2], float (&l)[2],
+                                                   float (&acc)[HDV / 8][4]) {
     constexpr int NKEYS = DK_PAGE;
     const int lane = threadIdx.x & 31, t = lane & 3;
     float s[NKEYS / 8][4];
@@ -71,7 +76,7 @@ __device__ __forceinline__ void warp_attend_masked(const uint32_t (&qf)[HD / 16]
             const int key = key0 + nt * 8 + 2 * t + (c & 1), r = c >> 1;
             float v = -INFINITY;
             if (key >= lo[r] && key <= hi[r]) {
-                v = s[nt][c] * sl2;
+                v = cap2 > 0.f ? cap2 * capped_unit(s[nt][c] * cap_in) : s[nt][c] * sl2;
                 if (b1 != 0.f) v -= b1 * __log2f(fmaf(b2, (float)(hi[r] - key), 1.f));
             }
             s[nt][c] = v;
@@ -137,8 +142,8 @@ __global__ void __launch_bounds__(128)
 attn_masked_prefill_kernel(const bf16* q, long long ldq, bf16* out, long long ldo, const bf16* gate, long long ldg,
                            float out_scale, const bf16* k_store, const bf16* v_store, const int* tiles, const int* cu_q,
                            const int* seq_pos0, const int* page_table, int pt_stride, int nh, int nkv, int window,
-                           int chunk, float sl2, const float* __restrict__ r1, const float* __restrict__ r2,
-                           const float* __restrict__ sink) {
+                           int chunk, float sl2, float cap2, float cap_in, const float* __restrict__ r1,
+                           const float* __restrict__ r2, const float* __restrict__ sink) {
     extern __shared__ __align__(16) bf16 smem[];
     pdl_wait();
     pdl_launch_dependents();
@@ -187,7 +192,7 @@ attn_masked_prefill_kernel(const bf16* q, long long ldq, bf16* out, long long ld
         const int key0 = jt * DK_PAGE;
         if (key0 <= w_hi && key0 + DK_PAGE - 1 >= w_lo && warp * 16 < rows_here) {
             const bf16* Ks = smem + cur * MSTAGE;
-            warp_attend_masked(qf, Ks, Ks + KTILE, key0, lo, hi, sl2, b1, b2, m, l, acc);
+            warp_attend_masked(qf, Ks, Ks + KTILE, key0, lo, hi, sl2, cap2, cap_in, b1, b2, m, l, acc);
         }
         __syncthreads();
     }
@@ -236,7 +241,7 @@ constexpr int MD_RED_FLOATS = MD_THREADS * 4 * 8;
 __global__ void __launch_bounds__(MD_THREADS)
 attn_masked_decode_kernel(const bf16* q, long long ldq, bf16* out, long long ldo, const bf16* gate, long long ldg,
                           float out_scale, const bf16* k_store, const bf16* v_store, const int* row_pos,
-                          const int* page_table, int pt_stride, int nh, int nkv, int window, int chunk, float scale,
+                          const int* page_table, int pt_stride, int nh, int nkv, int window, int chunk, float scale, float cap,
                           const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
                           int span, const bf16* k_new, const bf16* v_new, long long ldkv, bf16* k_out, bf16* v_out,
                           int nsplit, float* ws_acc, float* ws_ml) {
@@ -303,6 +308,7 @@ attn_masked_decode_kernel(const bf16* q, long long ldq, bf16* out, long long ldo
                 if (gg < gn) {
                     const int h = kvh * G + g0 + gg;
                     float s = dot[gg] * scale;
+                    if (cap > 0.f) s = cap * tanhf(s / cap);
                     if (r1) s -= r1[h] * log1pf(r2[h] * (float)(pos - j));
                     sc[(g0 + gg) * span + jj] = s;
                 }
@@ -423,7 +429,7 @@ DK_EXPORT int dk_attn_masked_prefill_bf16(const void* q, long long ldq, void* ou
                                           long long ldg, float out_scale, const void* k_store, const void* v_store,
                                           const int* tiles, int n_tiles, const int* cu_q, const int* seq_pos0,
                                           const int* page_table, int pt_stride, int nh, int nkv, int window, int chunk,
-                                          float scale, const float* r1, const float* r2, const float* sink,
+                                          float scale, float softcap, const float* r1, const float* r2, const float* sink,
                                           cudaStream_t st) {
     if (nh % nkv != 0) return (int)cudaErrorInvalidValue;
     static bool attr = false;
@@ -433,8 +439,8 @@ DK_EXPORT int dk_attn_masked_prefill_bf16(const void* q, long long ldq, void* ou
     }
     return dk_launch(attn_masked_prefill_kernel, dim3(nh, n_tiles), dim3(128), MSMEM_BYTES, st, (const bf16*)q, ldq,
                      (bf16*)out, ldo, (const bf16*)gate, ldg, out_scale, (const bf16*)k_store, (const bf16*)v_store, tiles,
-                     cu_q, seq_pos0, page_table, pt_stride, nh, nkv, window, chunk, scale * 1.4426950408889634f, r1, r2,
-                     sink);
+                     cu_q, seq_pos0, page_table, pt_stride, nh, nkv, window, chunk, scale * 1.4426950408889634f,
+                     softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, r1, r2, sink);
 }
 
 // k_new, v_new (or null): rows [n_rows, nkv*HD] / [n_rows, nkv*HDV] of the step's projection, ldkv elements apart,
@@ -445,7 +451,7 @@ DK_EXPORT int dk_attn_masked_prefill_bf16(const void* q, long long ldq, void* ou
 DK_EXPORT int dk_attn_masked_decode_bf16(const void* q, long long ldq, void* out, long long ldo, const void* gate,
                                          long long ldg, float out_scale, const void* k_store, const void* v_store,
                                          const int* row_pos, const int* page_table, int pt_stride, int n_rows, int nh,
-                                         int nkv, int window, int chunk, float scale, const float* r1, const float* r2,
+                                         int nkv, int window, int chunk, float scale, float softcap, const float* r1, const float* r2,
                                          const float* sink, int span, const void* k_new, const void* v_new, long long ldkv,
                                          int nsplit, float* ws_acc, float* ws_ml, cudaStream_t st) {
     if (nh % nkv != 0 || nsplit < 1 || (nsplit > 1 && (ws_acc == nullptr || ws_ml == nullptr))) return (int)cudaErrorInvalidValue;
@@ -459,7 +465,7 @@ DK_EXPORT int dk_attn_masked_decode_bf16(const void* q, long long ldq, void* out
     }
     int e = dk_launch(attn_masked_decode_kernel, dim3(nkv, n_rows, nsplit), dim3(MD_THREADS), smem, st, (const bf16*)q, ldq,
                       (bf16*)out, ldo, (const bf16*)gate, ldg, out_scale, (const bf16*)k_store, (const bf16*)v_store, row_pos,
-                      page_table, pt_stride, nh, nkv, window, chunk, scale, r1, r2, sink, span, (const bf16*)k_new,
+                      page_table, pt_stride, nh, nkv, window, chunk, scale, softcap, r1, r2, sink, span, (const bf16*)k_new,
                       (const bf16*)v_new, ldkv, (bf16*)k_store, (bf16*)v_store, nsplit, ws_acc, ws_ml);
     if (e != 0 || nsplit == 1) return e;
     return dk_launch(attn_masked_merge_kernel, dim3((n_rows * nh + 3) / 4), dim3(128), 0, st, (const float*)ws_acc,

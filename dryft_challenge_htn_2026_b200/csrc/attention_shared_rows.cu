@@ -3,7 +3,7 @@
 // low-rank latents with the keys' up projection moved to the query's side: rows of [latent | rotated part], hundreds
 // of numbers wide, far beyond what a warp can hold as fragments. Built once per pair of sizes with -DHD= -DHDV=
 // (HD a multiple of 16 up to 640, HDV a multiple of 32 up to 512 and at most HD). A chunk mask or a window bounds
-// the keys; scores, softmax and sums are float32, P is rounded to bfloat16 before P.V.
+// the keys, a sink may join a head's denominator; scores, softmax and sums are float32, P is rounded to bfloat16 before P.V.
 //
 // A block of 8 warps owns 64 rows of the (query, head of the group) plane of one sequence and one key/value head:
 // with G heads in a group, 64 / G consecutive queries with all their heads (G >= 64: one query and 64 of its heads).
@@ -130,8 +130,8 @@ __device__ __forceinline__ void sr_products(const bf16* qa, const bf16* kc, cons
 __global__ void __launch_bounds__(SR_THREADS, 1)
 attn_shared_rows_kernel(const bf16* q, long long ldq, bf16* out, long long ldo, float out_scale, const bf16* k_store,
                         const int* tiles, const int* cu_q, const int* seq_pos0, const int* row_pos, const int* page_table,
-                        int pt_stride, int nh, int nkv, int window, int chunk, float sl2, int nsplit, float* ws_acc,
-                        float* ws_ml) {
+                        int pt_stride, int nh, int nkv, int window, int chunk, float sl2, const float* __restrict__ sink, int nsplit,
+                        float* ws_acc, float* ws_ml) {
     extern __shared__ __align__(16) bf16 smem[];
     bf16* Qs = smem;
     bf16* Ks = Qs + SR_Q_ELEMS;
@@ -288,7 +288,11 @@ attn_shared_rows_kernel(const bf16* q, long long ldq, bf16* out, long long ldo, 
             continue;
         }
         if (head[r] < 0) continue;
-        const float inv = lt > 0.f ? out_scale / lt : 0.f;
+        float inv = lt > 0.f ? out_scale / lt : 0.f;
+        if (sink != nullptr && lt > 0.f) {        // one more term of the denominator, in the log2 domain like the scores
+            const float s2 = sink[head[r]] * 1.4426950408889634f, top = fmaxf(m[r], s2), w = exp2f(m[r] - top);
+            inv = out_scale * w / (lt * w + exp2f(s2 - top));
+        }
         bf16* o = out + flat[r] * ldo + (size_t)head[r] * HDV + wc * SR_HALF + 2 * t;
 #pragma unroll
         for (int nt = 0; nt < SR_HALF / 8; nt++)
@@ -311,11 +315,11 @@ attn_shared_rows_kernel(const bf16* q, long long ldq, bf16* out, long long ldo, 
 }
 
 // The parts of a split step put together: a block per (row, head), a thread per four value columns. M = the parts'
-// largest maximum, w_s = 2^(m_s - M), L = sum_s l_s w_s, out = sum_s acc_s w_s / L * out_scale (maxima in the log2 domain).
+// largest maximum, w_s = 2^(m_s - M), L = sum_s l_s w_s (+ 2^(sink - M), the sink counting in M too), out = sum_s acc_s w_s / L * out_scale (maxima in the log2 domain).
 constexpr int SR_MAX_SPLITS = 16;
 __global__ void __launch_bounds__(HDV / 4)
 attn_shared_rows_merge_kernel(const float* __restrict__ ws_acc, const float* __restrict__ ws_ml, bf16* out, long long ldo,
-                              float out_scale, int nh, int nsplit) {
+                              float out_scale, const float* __restrict__ sink, int nh, int nsplit) {
     pdl_wait();
     pdl_launch_dependents();
     const int b = blockIdx.x / nh, h = blockIdx.x % nh;
@@ -326,6 +330,11 @@ attn_shared_rows_merge_kernel(const float* __restrict__ ws_acc, const float* __r
 #pragma unroll
     for (int s = 0; s < SR_MAX_SPLITS; s++)
         if (s < nsplit) M = fmaxf(M, ml[2 * s]);
+    if (sink != nullptr && M != -INFINITY) {      // a padding row (no part counts) stays zero
+        const float s2 = sink[h] * 1.4426950408889634f;
+        M = fmaxf(M, s2);
+        L = exp2f(s2 - M);
+    }
 #pragma unroll
     for (int s = 0; s < SR_MAX_SPLITS; s++) {
         w[s] = (s < nsplit && M != -INFINITY) ? exp2f(ml[2 * s] - M) : 0.f;
@@ -350,8 +359,8 @@ attn_shared_rows_merge_kernel(const float* __restrict__ ws_acc, const float* __r
 DK_EXPORT int dk_attn_shared_rows_bf16(const void* q, long long ldq, void* out, long long ldo, float out_scale,
                                        const void* k_store, const int* tiles, int n_items, const int* cu_q,
                                        const int* seq_pos0, const int* row_pos, const int* page_table, int pt_stride,
-                                       int nh, int nkv, int window, int chunk, float scale, int nsplit, float* ws_acc,
-                                       float* ws_ml, cudaStream_t st) {
+                                       int nh, int nkv, int window, int chunk, float scale, const float* sink, int nsplit,
+                                       float* ws_acc, float* ws_ml, cudaStream_t st) {
     if (nh % nkv != 0 || nsplit < 1 || nsplit > SR_MAX_SPLITS || (nsplit > 1 && (tiles != nullptr || ws_acc == nullptr || ws_ml == nullptr)))
         return (int)cudaErrorInvalidValue;
     if (ldq % 8 != 0 || ldo % 2 != 0 || ((uintptr_t)q & 15) != 0 || ((uintptr_t)out & 3) != 0) return (int)cudaErrorInvalidValue;
@@ -363,10 +372,10 @@ DK_EXPORT int dk_attn_shared_rows_bf16(const void* q, long long ldq, void* out, 
     const int G = nh / nkv, HB = (G + SR_ROWS - 1) / SR_ROWS;
     int e = dk_launch(attn_shared_rows_kernel, dim3(n_items, nkv * HB, nsplit), dim3(SR_THREADS), SR_SMEM_BYTES, st,
                       (const bf16*)q, ldq, (bf16*)out, ldo, out_scale, (const bf16*)k_store, tiles, cu_q, seq_pos0, row_pos,
-                      page_table, pt_stride, nh, nkv, window, chunk, scale * 1.4426950408889634f, nsplit, ws_acc, ws_ml);
+                      page_table, pt_stride, nh, nkv, window, chunk, scale * 1.4426950408889634f, sink, nsplit, ws_acc, ws_ml);
     if (e != 0 || nsplit == 1) return e;
     return dk_launch(attn_shared_rows_merge_kernel, dim3(n_items * nh), dim3(HDV / 4), 0, st, (const float*)ws_acc,
-                     (const float*)ws_ml, (bf16*)out, ldo, out_scale, nh, nsplit);
+                     (const float*)ws_ml, (bf16*)out, ldo, out_scale, sink, nh, nsplit);
 }
 
 DK_EXPORT int dk_attn_shared_rows_tile_queries(int group) { return max(1, SR_ROWS / min(group, SR_ROWS)); }

@@ -50,8 +50,10 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 
 // xIELU: f(z) = ap z^2 + z/2 for z > 0, an (e^z - 1 - z) + z/2 otherwise (ap, an > 0 are made on the host from the two
-// learned numbers); arithmetic in float32. The row kernel and the epilogues of the three products share it.
+// learned numbers); arithmetic in float32. The row kernel and the epilogues of the three products share it. A negative an
+// selects the squared ReLU instead: f(z) = ap max(z, 0)^2.
 __device__ __forceinline__ float xielu_f(float z, float ap, float an) {
+    if (an < 0.f) return z > 0.f ? ap * z * z : 0.f;
     return z > 0.f ? fmaf(ap * z, z, 0.5f * z) : fmaf(an, expm1f(z) - z, 0.5f * z);
 }
 

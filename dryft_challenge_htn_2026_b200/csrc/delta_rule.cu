@@ -1,0 +1,389 @@
+// The gated delta rule over a float32 state per (sequence, head), S [D, V]:
+//     S <- g_t S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
+// with unit keys and queries shared by the heads of a group, one decay g and one step size beta per head and token.
+//   * delta_prepare  : what enters the recurrence, in float32, from the projection's rows: a causal convolution per channel
+//                      of q, k and v (its memory, the last taps - 1 projected rows, is a per-sequence state, read only
+//                      here), SiLU; q and k over sqrt(sum of squares + unit_eps) per head, q times D^(-1/2); g = exp(-exp(A)
+//                      softplus(a + dt)), beta = sigmoid(b); and k . q per key head (below).
+//   * delta_rule     : portions. One reduction over the state's rows a token: with a = S^T k and b = S^T q of the state as
+//                      the token finds it, u = beta (v - g a) and o = g b + (k . q) u. Eight lanes share a column of the
+//                      state, each with D / 8 of its rows in registers for the whole portion; the rows q, k, v of 16 tokens
+//                      at a time come through shared memory by cp.async, three chunks in turn.
+//   * delta_rule_step: one token a sequence: a block per (sequence, head, 32 columns) passes once over its part of the state.
+// Rows with position < 0 are padding: zeros out, states untouched.
+#include "common.cuh"
+
+#define DP_THREADS 256
+#define DR_NT 16            // tokens a staged chunk
+#define DR_STAGES 3
+#define DR_WARPS 4
+#define DR_COLS (4 * DR_WARPS)
+
+__device__ __forceinline__ float dr_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+
+template <typename T> __device__ __forceinline__ void dr_ld4(const T* p, float (&y)[4]);
+template <> __device__ __forceinline__ void dr_ld4<float>(const float* p, float (&y)[4]) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    y[0] = x.x, y[1] = x.y, y[2] = x.z, y[3] = x.w;
+}
+template <> __device__ __forceinline__ void dr_ld4<bf16>(const bf16* p, float (&y)[4]) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+    y[0] = a.x, y[1] = a.y, y[2] = b.x, y[3] = b.y;
+}
+
+// A block per token. proj rows [q (G D) | k (G D) | v (H V)]; a_rows, b_rows: columns [H] of the same matrix (row stride ld).
+// qkv [rows, 2 G D + H V] float32 out; scal [rows, 2 H + G] float32 out: g, beta, k . q.
+template <typename T>
+__global__ void __launch_bounds__(DP_THREADS)
+delta_prepare_kernel(const T* proj, long long ld, const T* a_rows, const T* b_rows, const T* state, const T* __restrict__ wconv,
+                     int taps, const float* __restrict__ a_log, const float* __restrict__ dt_bias, float unit_eps, const int* row_pos,
+                     const int* row_seq, const int* seq_pos0, const int* seq_slot, float* qkv, float* scal, int H, int G, int D, int V,
+                     int vec) {
+    extern __shared__ __align__(16) float row[];         // [C] after convolution and SiLU
+    pdl_wait();
+    pdl_launch_dependents();
+    const int nqk = G * D, C = 2 * nqk + H * V, t = blockIdx.x, tid = threadIdx.x;
+    float* out = qkv + (size_t)t * C;
+    float* sc = scal + (size_t)t * (2 * H + G);
+    const int pos = row_pos[t];
+    if (pos < 0) {
+        for (int c = tid; c < C; c += DP_THREADS) out[c] = 0.f;
+        for (int c = tid; c < 2 * H + G; c += DP_THREADS) sc[c] = 0.f;
+        return;
+    }
+    const int s = row_seq[t], p0 = seq_pos0[s];
+    const T* st = taps > 1 ? state + (size_t)seq_slot[s] * (taps - 1) * C : nullptr;
+    if (vec) {
+        for (int c = 4 * tid; c < C; c += 4 * DP_THREADS) {
+            float acc[4] = {0.f, 0.f, 0.f, 0.f};
+            float w[4][4];
+            if (taps == 4) {
+#pragma unroll
+                for (int e = 0; e < 4; e++) dr_ld4<T>(wconv + (size_t)(c + e) * 4, w[e]);
+            }
+            auto tap = [&](int j, float w0, float w1, float w2, float w3) {
+                const int back = taps - 1 - j, pp = pos - back;
+                float u[4];
+                dr_ld4<T>(pp >= p0 ? proj + (size_t)(t - back) * ld + c : st + (size_t)(taps - 1 - (p0 - pp)) * C + c, u);
+                acc[0] = fmaf(w0, u[0], acc[0]), acc[1] = fmaf(w1, u[1], acc[1]);
+                acc[2] = fmaf(w2, u[2], acc[2]), acc[3] = fmaf(w3, u[3], acc[3]);
+            };
+            if (taps == 4) {
+#pragma unroll
+                for (int j = 0; j < 4; j++) tap(j, w[0][j], w[1][j], w[2][j], w[3][j]);
+            } else {
+                const T* wc = wconv + (size_t)c * taps;
+                for (int j = 0; j < taps; j++) tap(j, to_f(wc[j]), to_f(wc[taps + j]), to_f(wc[2 * taps + j]), to_f(wc[3 * taps + j]));
+            }
+            float y[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) y[e] = acc[e] * dr_sigmoid(acc[e]);
+            if (c < 2 * nqk) *reinterpret_cast<float4*>(row + c) = make_float4(y[0], y[1], y[2], y[3]);
+            else *reinterpret_cast<float4*>(out + c) = make_float4(y[0], y[1], y[2], y[3]);
+        }
+    } else {
+        for (int c = tid; c < C; c += DP_THREADS) {
+            float acc = 0.f;
+            for (int j = 0; j < taps; j++) {
+                const int back = taps - 1 - j, pp = pos - back;
+                const float u = to_f(pp >= p0 ? proj[(size_t)(t - back) * ld + c] : st[(size_t)(taps - 1 - (p0 - pp)) * C + c]);
+                acc = fmaf(to_f(wconv[(size_t)c * taps + j]), u, acc);
+            }
+            const float y = acc * dr_sigmoid(acc);
+            if (c < 2 * nqk) row[c] = y;
+            else out[c] = y;
+        }
+    }
+    for (int h = tid; h < H; h += DP_THREADS) {
+        const float z = to_f(a_rows[(size_t)t * ld + h]) + dt_bias[h];
+        const float dt = z > 20.f ? z : log1pf(expf(z));
+        sc[h] = expf(-expf(a_log[h]) * dt);
+        sc[H + h] = dr_sigmoid(to_f(b_rows[(size_t)t * ld + h]));
+    }
+    __syncthreads();
+    const int lane = tid & 31, warp = tid >> 5;
+    const float qs = 1.f / sqrtf((float)D);
+    for (int g = warp; g < G; g += DP_THREADS / 32) {
+        const float *q = row + g * D, *k = row + nqk + g * D;
+        float sq = 0.f, sk = 0.f, kq = 0.f;
+        for (int d = lane; d < D; d += 32) sq += q[d] * q[d], sk += k[d] * k[d];
+        const float rq = qs / sqrtf(warp_sum(sq) + unit_eps), rk = 1.f / sqrtf(warp_sum(sk) + unit_eps);
+        for (int d = lane; d < D; d += 32) {
+            const float a = q[d] * rq, b = k[d] * rk;
+            out[g * D + d] = a;
+            out[nqk + g * D + d] = b;
+            kq = fmaf(a, b, kq);
+        }
+        kq = warp_sum(kq);
+        if (lane == 0) sc[2 * H + g] = kq;
+    }
+}
+
+__device__ __forceinline__ void dr_cp(float* smem, const float* gmem, bool wide) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
+    if (wide) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(gmem) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(a), "l"(gmem) : "memory");
+}
+
+// grid (sequences, heads, ceil(V / 16)), 4 warps of 4 columns. RPL: rows of the state a lane holds, D <= 8 RPL. Lane i of the
+// eight that share a column holds rows 4 i + 32 j + (0 .. 3).
+template <int RPL>
+__global__ void __launch_bounds__(32 * DR_WARPS)
+delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state, const int* cu_q, const int* seq_pos0,
+                  const int* seq_slot, int H, int G, int D, int V, int wide_qk, int wide_v) {
+    constexpr int DP = 8 * RPL, NJ = RPL / 4;
+    constexpr int STAGE = DR_NT * (2 * DP + DR_COLS + 4);          // k, q, v columns, (g, beta, k . q, -)
+    extern __shared__ __align__(16) float dr_smem[];
+    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DR_COLS, kh = h / (H / G);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, i8 = lane & 7;
+    const int col = col0 + warp * 4 + (lane >> 3);
+    for (int i = tid; i < DR_STAGES * STAGE; i += 32 * DR_WARPS) dr_smem[i] = 0.f;      // rows past D stay zero
+    pdl_wait();
+    pdl_launch_dependents();
+    if (seq_pos0[s] < 0) return;
+    const int r0 = cu_q[s], n_tok = cu_q[s + 1] - r0;
+    const int C = 2 * G * D + H * V, nsc = 2 * H + G;
+    const size_t ow = (size_t)H * V;
+    __syncthreads();
+    const int n_cols = min(DR_COLS, V - col0);
+    auto fetch = [&](int c) {                     // chunk c into its stage
+        float* base = dr_smem + (c % DR_STAGES) * STAGE;
+        const int t0 = c * DR_NT, nt = min(DR_NT, n_tok - t0);
+        const float* src = qkv + (size_t)(r0 + t0) * C;
+        const int step = wide_qk ? 4 : 1, per = D / step;
+        for (int i = tid; i < 2 * nt * per; i += 32 * DR_WARPS) {
+            const int which = i / (nt * per), tt = i / per % nt, d = (i % per) * step;      // 0: k, 1: q
+            dr_cp(base + which * DR_NT * DP + tt * DP + d, src + (size_t)tt * C + (which ? 0 : G * D) + kh * D + d, wide_qk);
+        }
+        const int vstep = wide_v ? 4 : 1, vper = n_cols / vstep;
+        for (int i = tid; i < nt * vper; i += 32 * DR_WARPS) {
+            const int tt = i / vper, d = (i % vper) * vstep;
+            dr_cp(base + 2 * DR_NT * DP + tt * DR_COLS + d, src + (size_t)tt * C + 2 * G * D + h * V + col0 + d, wide_v);
+        }
+        float* sc = base + DR_NT * (2 * DP + DR_COLS);
+        for (int i = tid; i < nt * 3; i += 32 * DR_WARPS) {
+            const int tt = i / 3, w = i % 3;
+            dr_cp(sc + tt * 4 + w, scal + (size_t)(r0 + t0 + tt) * nsc + (w == 0 ? h : w == 1 ? H + h : 2 * H + kh), false);
+        }
+    };
+    const int n_chunks = (n_tok + DR_NT - 1) / DR_NT;
+#pragma unroll
+    for (int c = 0; c < DR_STAGES - 1; c++) {
+        if (c < n_chunks) fetch(c);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    const bool live = col < V;
+    float* S = state + (((size_t)seq_slot[s] * H + h) * D) * V + col;
+    float st[RPL];
+#pragma unroll
+    for (int j = 0; j < NJ; j++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int d = 4 * i8 + 32 * j + e;
+            st[4 * j + e] = live && d < D ? S[(size_t)d * V] : 0.f;
+        }
+    for (int c = 0; c < n_chunks; c++) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(DR_STAGES - 2) : "memory");
+        __syncthreads();                           // chunk c is there, and every warp has left chunk c - 1
+        if (c + DR_STAGES - 1 < n_chunks) fetch(c + DR_STAGES - 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        const float* base = dr_smem + (c % DR_STAGES) * STAGE;
+        const float *ks = base + 4 * i8, *qs = ks + DR_NT * DP;
+        const float* vs = base + 2 * DR_NT * DP + warp * 4 + (lane >> 3);
+        const float4* scs = reinterpret_cast<const float4*>(base + DR_NT * (2 * DP + DR_COLS));
+        const int nt = min(DR_NT, n_tok - c * DR_NT);
+        float kn[RPL], qn[RPL];
+        auto rows_of = [&](int tt) {
+#pragma unroll
+            for (int j = 0; j < NJ; j++) {
+                const float4 x = *reinterpret_cast<const float4*>(ks + tt * DP + 32 * j);
+                const float4 y = *reinterpret_cast<const float4*>(qs + tt * DP + 32 * j);
+                kn[4 * j] = x.x, kn[4 * j + 1] = x.y, kn[4 * j + 2] = x.z, kn[4 * j + 3] = x.w;
+                qn[4 * j] = y.x, qn[4 * j + 1] = y.y, qn[4 * j + 2] = y.z, qn[4 * j + 3] = y.w;
+            }
+        };
+        rows_of(0);
+        for (int tt = 0; tt < nt; tt++) {
+            float kv[RPL], qv[RPL];
+#pragma unroll
+            for (int j = 0; j < RPL; j++) kv[j] = kn[j], qv[j] = qn[j];
+            const float4 g4 = scs[tt];
+            const float v = vs[tt * DR_COLS];
+            rows_of(min(tt + 1, nt - 1));
+            float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < RPL; j++) {
+                a[j & 3] = fmaf(st[j], kv[j], a[j & 3]);
+                b[j & 3] = fmaf(st[j], qv[j], b[j & 3]);
+            }
+            float as = (a[0] + a[1]) + (a[2] + a[3]), bs = (b[0] + b[1]) + (b[2] + b[3]);
+#pragma unroll
+            for (int off = 1; off < 8; off <<= 1) {
+                as += __shfl_xor_sync(0xffffffffu, as, off);
+                bs += __shfl_xor_sync(0xffffffffu, bs, off);
+            }
+            const float u = g4.y * (v - g4.x * as);
+#pragma unroll
+            for (int j = 0; j < RPL; j++) st[j] = fmaf(kv[j], u, g4.x * st[j]);
+            if (i8 == 0 && live) out[(size_t)(r0 + c * DR_NT + tt) * ow + (size_t)h * V + col] = fmaf(g4.z, u, g4.x * bs);
+        }
+    }
+    if (live) {
+#pragma unroll
+        for (int j = 0; j < NJ; j++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int d = 4 * i8 + 32 * j + e;
+                if (d < D) S[(size_t)d * V] = st[4 * j + e];
+            }
+    }
+}
+
+// One token a row: grid (rows, heads, ceil(V / 32)), 256 threads; thread (rg, c4): columns 4 c4 .. + 3 of the block's 32, state
+// rows rg, rg + 32, .. NR: rows a thread holds, D <= 32 NR. VEC: 16-byte accesses (V a multiple of 4).
+template <int NR, bool VEC>
+__global__ void __launch_bounds__(256)
+delta_rule_step_kernel(const float* qkv, const float* scal, float* out, float* state, const int* row_pos, const int* seq_slot, int H,
+                       int G, int D, int V) {
+    __shared__ float ks[256], qs[256];
+    __shared__ float4 red[8][8][2];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int r = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int c4 = tid & 7, rg = tid >> 3, col = blockIdx.z * 32 + 4 * c4, kh = h / (H / G);
+    const int C = 2 * G * D + H * V, nsc = 2 * H + G;
+    if (row_pos[r] < 0) {
+        if (rg == 0)
+            for (int e = 0; e < 4; e++)
+                if (col + e < V) out[(size_t)r * H * V + (size_t)h * V + col + e] = 0.f;
+        return;
+    }
+    const float* src = qkv + (size_t)r * C;
+    float* S = state + (((size_t)seq_slot[r] * H + h) * D) * V;
+    float st[NR][4];
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int d = rg + 32 * i;
+        if (VEC) {
+            const float4 x = d < D && col < V ? *reinterpret_cast<const float4*>(S + (size_t)d * V + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+            st[i][0] = x.x, st[i][1] = x.y, st[i][2] = x.z, st[i][3] = x.w;
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; e++) st[i][e] = d < D && col + e < V ? S[(size_t)d * V + col + e] : 0.f;
+        }
+    }
+    for (int d = tid; d < D; d += 256) qs[d] = src[kh * D + d], ks[d] = src[G * D + kh * D + d];
+    const float* sc = scal + (size_t)r * nsc;
+    const float g = sc[h], beta = sc[H + h], kq = sc[2 * H + kh];
+    float v[4];
+#pragma unroll
+    for (int e = 0; e < 4; e++) v[e] = col + e < V ? src[2 * G * D + h * V + col + e] : 0.f;
+    __syncthreads();
+    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int d = rg + 32 * i;
+        if (d < D) {
+            const float k = ks[d], q = qs[d];
+#pragma unroll
+            for (int e = 0; e < 4; e++) a[e] = fmaf(st[i][e], k, a[e]), b[e] = fmaf(st[i][e], q, b[e]);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        a[e] += __shfl_xor_sync(0xffffffffu, a[e], 8);
+        b[e] += __shfl_xor_sync(0xffffffffu, b[e], 8);
+        a[e] += __shfl_xor_sync(0xffffffffu, a[e], 16);
+        b[e] += __shfl_xor_sync(0xffffffffu, b[e], 16);
+    }
+    if (lane < 8) red[warp][c4][0] = make_float4(a[0], a[1], a[2], a[3]), red[warp][c4][1] = make_float4(b[0], b[1], b[2], b[3]);
+    __syncthreads();
+    float4 as = red[0][c4][0], bs = red[0][c4][1];
+#pragma unroll
+    for (int w = 1; w < 8; w++) {
+        const float4 x = red[w][c4][0], y = red[w][c4][1];
+        as.x += x.x, as.y += x.y, as.z += x.z, as.w += x.w;
+        bs.x += y.x, bs.y += y.y, bs.z += y.z, bs.w += y.w;
+    }
+    const float at[4] = {as.x, as.y, as.z, as.w}, bt[4] = {bs.x, bs.y, bs.z, bs.w};
+    float u[4];
+#pragma unroll
+    for (int e = 0; e < 4; e++) u[e] = beta * (v[e] - g * at[e]);
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int d = rg + 32 * i;
+        if (d >= D) continue;
+        const float k = ks[d];
+        if (VEC) {
+            if (col < V)
+                *reinterpret_cast<float4*>(S + (size_t)d * V + col) =
+                    make_float4(fmaf(k, u[0], g * st[i][0]), fmaf(k, u[1], g * st[i][1]), fmaf(k, u[2], g * st[i][2]), fmaf(k, u[3], g * st[i][3]));
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; e++)
+                if (col + e < V) S[(size_t)d * V + col + e] = fmaf(k, u[e], g * st[i][e]);
+        }
+    }
+    if (rg == 0)
+#pragma unroll
+        for (int e = 0; e < 4; e++)
+            if (col + e < V) out[(size_t)r * H * V + (size_t)h * V + col + e] = fmaf(kq, u[e], g * bt[e]);
+}
+
+DK_EXPORT int dk_delta_prepare(int dtype, const void* proj, long long ld, const void* a_rows, const void* b_rows, const void* state,
+                               const void* wconv, int taps, const float* a_log, const float* dt_bias, float unit_eps,
+                               const int* row_pos, const int* row_seq, const int* seq_pos0, const int* seq_slot, float* qkv,
+                               float* scal, int n_tok, int H, int G, int D, int V, cudaStream_t st) {
+    if (G < 1 || H % G || taps < 1 || (taps > 1 && state == nullptr)) return (int)cudaErrorInvalidValue;
+    const int C = 2 * G * D + H * V;
+    const size_t smem = sizeof(float) * (size_t)(2 * G * D);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    const int esz = dtype == 0 ? 4 : 2;
+    const int vec = C % 4 == 0 && (2 * G * D) % 4 == 0 && ld % 4 == 0 && (uintptr_t)qkv % 16 == 0 &&
+                    ((uintptr_t)proj | (uintptr_t)state | (uintptr_t)wconv) % (4 * esz) == 0;
+    if (dtype == 0) {
+        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        return dk_launch(delta_prepare_kernel<float>, dim3(n_tok), dim3(DP_THREADS), smem, st, (const float*)proj, ld,
+                         (const float*)a_rows, (const float*)b_rows, (const float*)state, (const float*)wconv, taps, a_log, dt_bias,
+                         unit_eps, row_pos, row_seq, seq_pos0, seq_slot, qkv, scal, H, G, D, V, vec);
+    }
+    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return dk_launch(delta_prepare_kernel<bf16>, dim3(n_tok), dim3(DP_THREADS), smem, st, (const bf16*)proj, ld, (const bf16*)a_rows,
+                     (const bf16*)b_rows, (const bf16*)state, (const bf16*)wconv, taps, a_log, dt_bias, unit_eps, row_pos, row_seq,
+                     seq_pos0, seq_slot, qkv, scal, H, G, D, V, vec);
+}
+
+DK_EXPORT int dk_delta_rule(const float* qkv, const float* scal, float* out, float* state, const int* cu_q, const int* seq_pos0,
+                            const int* seq_slot, int n_seq, int H, int G, int D, int V, cudaStream_t st) {
+    if (G < 1 || H % G || D < 1 || D > 256 || V < 1 || cu_q == nullptr) return (int)cudaErrorInvalidValue;
+    const int C = 2 * G * D + H * V;
+    const int wide_qk = D % 4 == 0 && C % 4 == 0 && (uintptr_t)qkv % 16 == 0;
+    const int wide_v = wide_qk && V % 4 == 0;
+    const dim3 grid(n_seq, H, (V + DR_COLS - 1) / DR_COLS), block(32 * DR_WARPS);
+#define DR_LAUNCH(R)                                                                                                           \
+    if (D <= 8 * R) {                                                                                                          \
+        const size_t smem = sizeof(float) * DR_STAGES * DR_NT * (2 * 8 * R + DR_COLS + 4);                                     \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_rule_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        return dk_launch(delta_rule_kernel<R>, grid, block, smem, st, qkv, scal, out, state, cu_q, seq_pos0, seq_slot, H, G, D, V, \
+                         wide_qk, wide_v);                                                                                     \
+    }
+    DR_LAUNCH(4) DR_LAUNCH(8) DR_LAUNCH(16) DR_LAUNCH(32)
+#undef DR_LAUNCH
+    return (int)cudaErrorInvalidValue;
+}
+
+DK_EXPORT int dk_delta_rule_step(const float* qkv, const float* scal, float* out, float* state, const int* row_pos,
+                                 const int* seq_slot, int n_rows, int H, int G, int D, int V, cudaStream_t st) {
+    if (G < 1 || H % G || D < 1 || D > 256 || V < 1) return (int)cudaErrorInvalidValue;
+    const bool vec = V % 4 == 0 && (uintptr_t)state % 16 == 0;
+    const dim3 grid(n_rows, H, (V + 31) / 32), block(256);
+#define DS_LAUNCH(R)                                                                                                           \
+    if (D <= 32 * R)                                                                                                           \
+        return vec ? dk_launch(delta_rule_step_kernel<R, true>, grid, block, 0, st, qkv, scal, out, state, row_pos, seq_slot, H, G, D, V) \
+                   : dk_launch(delta_rule_step_kernel<R, false>, grid, block, 0, st, qkv, scal, out, state, row_pos, seq_slot, H, G, D, V);
+    DS_LAUNCH(1) DS_LAUNCH(2) DS_LAUNCH(4) DS_LAUNCH(8)
+#undef DS_LAUNCH
+    return (int)cudaErrorInvalidValue;
+}

@@ -3,7 +3,8 @@
 // latent, r (rot_dim) the one rotated key part that all heads share.
 //   latent_norm_rope_write : c_q = rmsnorm(a) * w_q -> dense rows; c = rmsnorm(b) * w_kv and r rotated by pairs
 //                            -> the token's place in the paged cache: key row [c | r] (one kv head), whose first kv_rank
-//                            numbers are the value row (a cache with a store of values gets c there as well).
+//                            numbers are the value row (a cache with a store of values gets c there as well). q_rank 0:
+//                            rows [b | r], no query latent.
 //   latent_query           : per (token, head) the query of the up projection [plain (dim) | rot (rot_dim)] becomes
 //                            [W_uk_h^T plain (kv_rank) | rot rotated by pairs]: the plain key's up projection moved to
 //                            the query's side, so that scores are taken against the cached latent itself.
@@ -28,7 +29,7 @@ latent_norm_rope_write_kernel(const T* proj, long long ld, T* cq_out, long long 
     const int pos = row_pos[t];
     if (pos < 0) return;
     const T* row = proj + (size_t)t * ld;
-    if (blockIdx.y == 0) {                    // the query latent
+    if (blockIdx.y == 1) {                    // the query latent (a second block, only where there is one)
         float ss = 0.f;
         for (int i = threadIdx.x; i < q_rank; i += LT_THREADS) {
             const float v = to_f(row[i]);
@@ -168,7 +169,7 @@ DK_EXPORT int dk_latent_norm_rope_write(int dtype, const void* proj, long long l
                                         int q_rank, int kv_rank, int rot_dim, void* k_store, void* v_store,
                                         const int* page_table, int pt_stride, cudaStream_t st) {
     if (rot_dims % 2 || rot_dims > rot_dim) return (int)cudaErrorInvalidValue;
-    LT_DISPATCH(dtype, return dk_launch(latent_norm_rope_write_kernel<T>, dim3(n_tok, 2), dim3(LT_THREADS), 0, st,
+    LT_DISPATCH(dtype, return dk_launch(latent_norm_rope_write_kernel<T>, dim3(n_tok, q_rank > 0 ? 2 : 1), dim3(LT_THREADS), 0, st,
                                         (const T*)proj, ld, (T*)cq_out, ldq, wq, wkv, eps, cosv, sinv, rot_dims, row_pos,
                                         row_seq, q_rank, kv_rank, rot_dim, (T*)k_store, (T*)v_store, page_table, pt_stride));
 }

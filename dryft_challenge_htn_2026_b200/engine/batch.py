@@ -33,6 +33,17 @@ class StepContext:
         self.plans = {}
         self.host = None
 
+    def sequences(self):
+        """(cu_q, tokens cached before the step, sequences) as the kernels with a per-sequence state want them: in a decode
+        step no cu_q (row s is sequence s, its position is what came before; padding rows carry position -1)."""
+        if self.is_decode:
+            return None, self.row_pos, self.n_tok
+        return self.cu_q, self.seq_pos0, self.n_seq
+
+    def sequence_rows(self):
+        """(row_pos, row_seq, cu_q, seq_slot) for kernels that work row by row; cu_q None in a decode step."""
+        return self.row_pos, self.row_seq, None if self.is_decode else self.cu_q, self.seq_slot
+
     def scratch(self, key, make):
         """A buffer (or tuple of buffers) that lives as long as the runner and is reused by every
         step with the same key; kernels' scratch memory comes from here."""

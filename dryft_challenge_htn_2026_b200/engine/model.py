@@ -4,6 +4,7 @@ describes and returns float32 logits at the wanted rows (reference: engine/engin
 """
 import torch
 
+from ..cache.requests import StateRequest
 from ..csrc import api
 from ..parts import ParamDecl, Runtime, build_part
 from ..parts.block import add_norm
@@ -34,6 +35,11 @@ class CausalLM:
             if self.blocks[e.layer].cache_requests() != self.blocks[owners[e.cache]].cache_requests():
                 raise ValueError(f"layer {e.layer} cannot use cache entry {e.cache}: its owner stores something else")
         self._entry_requests = [self.blocks[owners[c]].cache_requests() for c in range(n_entries)]
+        self.bigram = None       # the table of token pairs (ModelSpec.embed_bigram); its memory is a cache entry behind the layers'
+        if spec.embed_bigram is not None:
+            if spec.embed_position is not None or any(e.add_embedding for e in spec.schedule):
+                raise ValueError("an embedding with token pairs goes without a position vector and is not taken in again")
+            self._entry_requests.append([StateRequest((1,), torch.int32)])
         self.embed = self.head = None
         self.tied = None
         self.position = build_part(spec.embed_position, self.rt) if spec.embed_position is not None else None
@@ -55,6 +61,9 @@ class CausalLM:
         """Checkpoint name -> ParamDecl for the whole model."""
         s = self.spec
         out = {s.embed_name: ParamDecl(s.embed_name, (s.vocab_size, s.hidden_size), "matrix")}
+        if s.embed_bigram is not None:
+            b = s.embed_bigram
+            out[b.tensor] = ParamDecl(b.tensor, (b.buckets + 1, s.hidden_size), "matrix")
         for ls, blk in zip(s.layers, self.blocks):
             for p in blk.param_decls():
                 out[ls.prefix + p.name] = p
@@ -71,6 +80,8 @@ class CausalLM:
         self.tied = tied
         self.embed = tensors.pop(s.embed_name).contiguous()
         self.head = self.embed if tied else tensors.pop(s.head_name).contiguous()
+        if s.embed_bigram is not None:
+            self.bigram = tensors.pop(s.embed_bigram.tensor).contiguous()
         self.tables = {name: tensors.pop(name).to(torch.float32).contiguous() for name, _ in s.tables}
         for ls, blk in zip(s.layers, self.blocks):
             n = len(ls.prefix)
@@ -115,7 +126,13 @@ class CausalLM:
         ctx.carry = {}           # what one layer of the step leaves for later ones (e.g. values that layers share)
         ctx.stream_copy = None   # the stream in the storage type, where a kernel has left it (blocks with the norm after the sum)
         plain = getattr(first, "reads_stream", False) and not (s.schedule[0].add_embedding or s.schedule[0].add_row)
-        if self.position is None and s.embed_scale == 1.0:
+        ctx.stream = None        # the stream, where a block has written it to another buffer than the one it was given
+        if self.bigram is not None:
+            b = s.embed_bigram
+            api.embed_bigram(ctx.tok, self.embed, s.embed_scale, self.bigram, b.mul_prev, b.mul_cur,
+                             cache.views(len(self._entry_requests) - 1)[0].state, ctx.sequence_rows(), h)
+            fused = False
+        elif self.position is None and s.embed_scale == 1.0:
             api.embed_rmsnorm(ctx.tok, self.embed, norm_w, eps, h, a if (fused or plain) else None)
             if plain:
                 ctx.stream_copy = a
@@ -131,6 +148,8 @@ class CausalLM:
                 ctx.stream_copy = None
             pending = self.blocks[e.layer].forward(ctx, h, pending, cache.views(e.cache), e.writes,
                                                    a if (i == 0 and fused) else None)
+            if ctx.stream is not None:
+                h, ctx.stream = ctx.stream, None
             if tap is not None:
                 tap(i, h.clone() if pending is None else
                     h + (pending.to_float32() if hasattr(pending, "to_float32") else

@@ -1,11 +1,11 @@
-"""Grouped-query softmax attention without rotation over the paged cache, with a chunk mask or a
+"""Grouped-query softmax attention over the paged cache, with a chunk mask or a
 window, a logarithmic distance bias, a sink in the softmax's denominator and an output gate, each
 switched on by its specification; key and value heads may differ in size.
 
 forward = one fused projection [q; k; v; gate] -> (where the specification asks: a short causal convolution
 over time on q, k and v with a per-sequence state, a norm per q and k head, a rotation of the heads' first
-coordinates; one kernel) -> k and v into the cache -> attention over the cache with the gate in its epilogue
--> output projection. Further options of the scores: a cap, first tokens that the window keeps, a sink fixed
+coordinates; one kernel; or q and k normed as whole projections, rotated by pairs, values turned by their position: another) -> k and v into the cache -> attention over the cache with the gate in its epilogue
+(a kernel behind it where turned values are turned back or each head has one gate) -> output projection. Further options of the scores: a cap, first tokens that the window keeps, a sink fixed
 at zero. Kernels: bfloat16 prompts with equal head sizes of 64
 or 128 on tcgen05 tensor cores, other head sizes in steps of 16 on mma.sync, single tokens by a kernel of
 their own, and float32 (or any other size) on the float32-arithmetic kernel that serves every phase. The part also runs as a branch of a
@@ -36,7 +36,12 @@ class MaskedAttention(Part):
             raise ValueError(f"values of {s.v_head_dim} numbers cannot be the start of key rows of {s.head_dim}")
         self.n_q, self.n_k = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
         self.n_v, self.n_mid = s.num_kv_heads * s.v_head_dim, s.num_heads * s.v_head_dim
-        self.n_in = self.n_q + self.n_k + self.n_v + (self.n_mid if s.output_gate else 0)
+        if s.head_gate and s.output_gate:
+            raise ValueError("a gate per head and a gate per coordinate exclude each other")
+        self.n_gate = self.n_mid if s.output_gate else s.num_heads if s.head_gate else 0
+        self.n_in = self.n_q + self.n_k + self.n_v + self.n_gate
+        if s.head_gate:      # a few gate rows behind q, k, v: filled up with zero rows, so that rows of the product stay aligned
+            self.n_in = (self.n_in + 7) // 8 * 8
         self.r1 = self.r2 = self.sink = None
         if s.unit_sink:
             if s.sink:
@@ -63,23 +68,34 @@ class MaskedAttention(Part):
                              f"up to {api.TALK_MAX_OUT}")
         if s.q_temp is not None and not (int(s.q_temp[1]) >= 1):
             raise ValueError(f"a query temperature every {s.q_temp[1]} positions")
+        # q and k normed as wholes, a rotation by pairs, values that turn: the row kernel without convolution and biases
+        self.value_position = build_part(s.value_position, rt) if s.value_position is not None else None
+        self.row_kernel = self.value_position is not None or s.qk_norm_whole or getattr(self.position, "pairs", False)
+        if self.row_kernel and (s.conv_taps not in (None, 1) or s.bias or s.q_temp is not None or s.value_mix is not None or s.talk):
+            raise ValueError("rotation by pairs, a norm of the whole projection and turning values go without a convolution, "
+                             "biases, a query temperature, blended values and mixed head scores")
+        if self.value_position is not None and self.value_position.spec.dim != s.v_head_dim:
+            raise ValueError(f"values of {s.v_head_dim} turned over {self.value_position.spec.dim} coordinates")
+        if s.qk_norm_whole and (s.qk_norm is None or s.norm_after_rotation):
+            raise ValueError("a norm of the whole projection stands before the rotation")
+        self.behind = self.value_position is not None or s.head_gate      # a row kernel follows the attention
         self.bias = self.talk = None
         self.prepares = self.taps > 1 or self.qk_norm is not None or self.position is not None or s.value_mix is not None \
-            or s.bias or s.q_temp is not None
+            or s.bias or s.q_temp is not None or self.row_kernel
         self.n_qkv = self.n_q + self.n_k + self.n_v
         self.q_norm_w = self.k_norm_w = self.w_conv = None
         self.max_positions = 0
         # the tensor-core kernels take bfloat16 with head sizes in steps of 16; everything else (float32, odd
         # head sizes) runs on the float32-arithmetic kernel, which serves every phase
         self.tensor_core = rt.dtype == torch.bfloat16 and api.masked_bf16_takes(s.head_dim, s.v_head_dim)
-        # a cap on the scores and kept first tokens are options of the float32-arithmetic kernel, of the tcgen05 prompt
-        # kernel and of the split single-token kernel (equal head sizes); the mma.sync kernels for other sizes lack them
-        self.plain_options = s.softcap is None and not s.keep_first
+        # kept first tokens are an option of the float32-arithmetic kernel, of the tcgen05 prompt kernel and of the split
+        # single-token kernel (equal head sizes); the mma.sync kernels for other sizes lack them
+        self.plain_options = not s.keep_first
         self.tiles = QueryTiles(api.MASKED_TILE_ROWS) if self.tensor_core else None
         # value rows that are the key rows' first numbers, of sizes beyond those kernels: all heads of a group in one
         # block over the key rows alone (prompts and single tokens)
         self.shared_rows = rt.dtype == torch.bfloat16 and not self.tensor_core and s.values_in_keys and self.plain_options \
-            and not (s.distance_bias or s.sink or s.unit_sink or s.output_gate) and api.shared_rows_takes(s.head_dim, s.v_head_dim)
+            and s.softcap is None and not (s.distance_bias or s.output_gate) and api.shared_rows_takes(s.head_dim, s.v_head_dim)
         self.row_tiles = QueryTiles(api.shared_rows_tile_queries(s.num_heads // s.num_kv_heads)) if self.shared_rows else None
         # equal head sizes of 64 or 128: prompts run on the tcgen05 kernel (its masked build), in tiles of 128 queries
         self.tc_tiles = QueryTiles(api.TC_TILE_ROWS) if self.tensor_core and s.head_dim == s.v_head_dim \
@@ -95,8 +111,8 @@ class MaskedAttention(Part):
         s = self.spec
         d = [ParamDecl("q", (self.n_q, s.hidden_size)), ParamDecl("k", (self.n_k, s.hidden_size)),
              ParamDecl("v", (self.n_v, s.hidden_size)), ParamDecl("o", (s.hidden_size, self.n_mid))]
-        if s.output_gate:
-            d.append(ParamDecl("g", (self.n_mid, s.hidden_size)))
+        if self.n_gate:
+            d.append(ParamDecl("g", (self.n_gate, s.hidden_size)))
         if s.distance_bias:
             d += [ParamDecl("r1", (s.num_heads,), init="positive", keep_float32=True),
                   ParamDecl("r2", (s.num_heads,), init="positive", keep_float32=True)]
@@ -106,8 +122,8 @@ class MaskedAttention(Part):
             d += [ParamDecl("q.conv", (self.n_q, self.taps), init="taps"), ParamDecl("k.conv", (self.n_k, self.taps), init="taps"),
                   ParamDecl("v.conv", (self.n_v, self.taps), init="taps")]
         if self.qk_norm_weights:
-            d += [ParamDecl("q.norm", (s.head_dim,), init="norm", keep_float32=True),
-                  ParamDecl("k.norm", (s.head_dim,), init="norm", keep_float32=True)]
+            d += [ParamDecl("q.norm", (self.n_q if s.qk_norm_whole else s.head_dim,), init="norm", keep_float32=True),
+                  ParamDecl("k.norm", (self.n_k if s.qk_norm_whole else s.head_dim,), init="norm", keep_float32=True)]
         if s.value_mix is not None:
             d.append(ParamDecl("vmix", (), init="fraction", keep_float32=True))
         if s.bias:
@@ -120,8 +136,11 @@ class MaskedAttention(Part):
 
     def bind(self, tensors):
         rows = [tensors.pop("q"), tensors.pop("k"), tensors.pop("v")]
-        if self.spec.output_gate:
+        if self.n_gate:
             rows.append(tensors.pop("g"))
+        fill = self.n_in - sum(w.shape[0] for w in rows)
+        if fill:
+            rows.append(torch.zeros((fill, self.spec.hidden_size), dtype=rows[0].dtype, device=rows[0].device))
         self.w_in = torch.cat(rows, 0).contiguous()
         self.w_o = tensors.pop("o").contiguous()
         if self.spec.distance_bias:
@@ -153,8 +172,29 @@ class MaskedAttention(Part):
 
     def prepare(self, max_positions):
         self.max_positions = max_positions
-        if self.position is not None:
-            self.position.tables(max_positions)
+        for pos in (self.position, self.value_position):
+            if pos is not None:
+                pos.tables(max_positions)
+
+    def _rotation(self, ctx, position):
+        """(cos, sin, dims, pairs) of a rotation part for the kernels, or None."""
+        if position is None:
+            return None
+        cos, sin = position.tables(max(self.max_positions, ctx.max_position + 1))
+        return cos, sin, position.spec.dim, getattr(position, "pairs", False)
+
+    def rotated_queries(self, ctx, views, proj, writes=True):
+        """q rows of the projection after norm and rotation; with ``writes`` the k and v heads, normed and turned, go into the
+        cache."""
+        s, kv = self.spec, views[0]
+        out = torch.empty((ctx.n_tok, self.n_q), dtype=self.rt.dtype, device=self.rt.device)
+        mode = api.NORM_NONE if self.qk_norm is None else api.NORM_WHOLE if s.qk_norm_whole else \
+            api.NORM_AFTER_ROTATION if s.norm_after_rotation else api.NORM_BEFORE_ROTATION
+        api.qkv_rows(proj[:, :self.n_qkv], out, mode, self.q_norm_w, self.k_norm_w, self.qk_norm.eps if self.qk_norm is not None else 0.0,
+                     self._rotation(ctx, self.position), self._rotation(ctx, self.value_position), ctx.row_pos, ctx.row_seq,
+                     s.num_heads, s.num_kv_heads, s.head_dim, s.v_head_dim, kv.k if writes else None, kv.v if writes else None,
+                     ctx.tables[kv.group] if writes else None)
+        return out
 
     def prepared_rows(self, ctx, views, proj, writes=True):
         """[q | k | v] of the projection rows after the convolution, the head norm and the rotation, as a dense
@@ -194,7 +234,17 @@ class MaskedAttention(Part):
         """``proj`` [tokens, n_in]: this part's rows of a projection (possibly columns of a wider matrix);
         ``mid`` [tokens, n_mid]: where scale * (gated heads) go."""
         s, kv = self.spec, views[0]
-        gate = proj[:, self.n_q + self.n_k + self.n_v:] if s.output_gate else None
+        gate = proj[:, self.n_qkv:self.n_qkv + self.n_gate] if self.n_gate else None
+        if self.row_kernel:
+            q = self.rotated_queries(ctx, views, proj, writes)
+            if not self.behind:
+                return self.attend(ctx, kv, q, None, None, gate, mid, scale, writes=False)
+            o = torch.empty((ctx.n_tok, self.n_mid), dtype=self.rt.dtype, device=self.rt.device)
+            self.attend(ctx, kv, q, None, None, None if s.head_gate else gate, o, 1.0, writes=False)
+            return api.turn_back_gate(o, mid, gate if s.head_gate else None, self._rotation(ctx, self.value_position), scale,
+                                      ctx.row_pos, s.num_heads, s.v_head_dim)
+        if s.head_gate:
+            raise ValueError("a gate per head without a rotation by pairs, a norm of the whole projection or turning values")
         if self.prepares:
             proj = self.prepared_rows(ctx, views, proj, writes)
             writes = False          # that kernel has stored the step's keys and values
@@ -245,18 +295,20 @@ class MaskedAttention(Part):
                 ws = ctx.scratch(("masked_decode", ctx.n_tok, s.num_heads, s.v_head_dim, span[1]),
                                  lambda: api.masked_decode_ws(ctx.n_tok, s.num_heads, s.v_head_dim, span[1], self.rt.device))
             return api.attention_masked_decode_bf16(q, mid, gate, scale, kv.k, kv.v, ctx.row_pos, table, *sizes, span,
-                                                    self.r1, self.r2, self.sink, k if writes else None, v if writes else None, ws)
+                                                    self.r1, self.r2, self.sink, k if writes else None, v if writes else None, ws,
+                                                    s.softcap)
         if writes:
             api.kv_write(k, v, kv.k, kv.v, ctx.row_pos, ctx.row_seq, table, s.num_kv_heads, s.head_dim, s.v_head_dim)
         if self.shared_rows and gate is None and api.shared_rows_operands(q, mid):
             if not ctx.is_decode:
                 return api.attention_shared_rows_bf16(q, mid, scale, kv.k, table, *sizes, tiles=ctx.plans[self.row_tiles.key],
-                                                      cu_q=ctx.cu_q, seq_pos0=ctx.seq_pos0)
+                                                      cu_q=ctx.cu_q, seq_pos0=ctx.seq_pos0, sink=self.sink)
             nsplit = api.shared_rows_splits(ctx.n_tok, s.num_heads, s.num_kv_heads, table.shape[1], s.window, s.chunk)
             ws = ctx.scratch(("shared_rows", ctx.n_tok, s.num_heads, s.v_head_dim, nsplit),
                              lambda: api.shared_rows_ws(ctx.n_tok, s.num_heads, s.v_head_dim, nsplit, self.rt.device)) \
                 if nsplit > 1 else None
-            return api.attention_shared_rows_bf16(q, mid, scale, kv.k, table, *sizes, row_pos=ctx.row_pos, nsplit=nsplit, ws=ws)
+            return api.attention_shared_rows_bf16(q, mid, scale, kv.k, table, *sizes, row_pos=ctx.row_pos, nsplit=nsplit, ws=ws,
+                                                  sink=self.sink)
         if self.tc_tiles is not None and not ctx.is_decode and api.masked_tc_takes(q, mid, gate, s.head_dim, s.v_head_dim):
             return api.attention_masked_prefill_tc(q, mid, gate, scale, kv.k, kv.v, ctx.plans[self.tc_tiles.key], ctx.cu_q,
                                                    ctx.seq_pos0, table, s.num_heads, s.num_kv_heads, s.head_dim, s.window,
@@ -264,7 +316,7 @@ class MaskedAttention(Part):
         even = all(t is None or (t.stride(0) % 2 == 0 and t.data_ptr() % 4 == 0) for t in (q, mid, gate))
         if self.tensor_core and self.plain_options and not ctx.is_decode and even:
             return api.attention_masked_prefill_bf16(q, mid, gate, scale, kv.k, kv.v, ctx.plans[self.tiles.key], ctx.cu_q,
-                                                     ctx.seq_pos0, table, *sizes, self.r1, self.r2, self.sink)
+                                                     ctx.seq_pos0, table, *sizes, self.r1, self.r2, self.sink, s.softcap)
         api.attention_masked(q, mid, gate, scale, kv.k, kv.v, ctx.row_pos, ctx.row_seq, table, *sizes, self.r1, self.r2,
                              self.sink, s.softcap, s.keep_first)
 

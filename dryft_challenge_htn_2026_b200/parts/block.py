@@ -8,10 +8,11 @@ norm that says ``takes_partial`` adds them up while it reads, for any other they
 """
 import torch
 
-from ..config.specs import LayerSpec, PostNormLayerSpec, SandwichLayerSpec
+from ..cache.requests import StateRequest
+from ..config.specs import LayerSpec, OutputNormLayerSpec, PostNormLayerSpec, SandwichLayerSpec
 from ..csrc import api
 from .base import ParamDecl, Part, build_part, register_part
-from .norm import NormedDelta, RMSNorm
+from .norm import NormedDelta, RMSNorm, norm_args
 
 
 class PreNormBlock(Part):
@@ -62,7 +63,7 @@ class PreNormBlock(Part):
 
 def add_norm(norm, h, delta, dtype, rows=None):
     """h += delta, then norm(h) (of the rows ``rows`` only, leaving h alone, when given)."""
-    if isinstance(delta, NormedDelta) and not isinstance(norm, RMSNorm):
+    if isinstance(delta, NormedDelta) and not isinstance(norm, RMSNorm) and not getattr(norm, "takes_normed", False):
         raise TypeError(f"{type(norm).__name__} cannot follow a sublayer whose output has a norm of its own")
     if isinstance(delta, api.Partial) and not getattr(norm, "takes_partial", False):
         delta = delta.sum(dtype)
@@ -154,3 +155,66 @@ class SandwichBlock(PreNormBlock):
 
 
 register_part(SandwichLayerSpec, SandwichBlock)
+
+
+class OutputNormBlock(PreNormBlock):
+    """A norm on each sublayer's output alone: h += norm_mix(mixer(h')); h += norm_ff(feed_forward(h)), with h' the stream, or
+    the stream mixed with that of the token before (``spec.shift``: a share per element; the vector of a sequence's last token
+    is per-sequence state in float32, the last of this block's cache requests). Like the other blocks it takes the block
+    before's output as ``pending`` and hands its own on, as a ``NormedDelta``; norm, sum and shift are one kernel, which
+    writes the stream to another buffer where there is a shift (``ctx.stream``)."""
+
+    def __init__(self, spec, rt):
+        Part.__init__(self, spec, rt)
+        self.mixer = build_part(spec.mixer, rt)
+        self.norm_mix = build_part(spec.norm_mix, rt)
+        self.feed_forward = build_part(spec.feed_forward, rt) if spec.feed_forward is not None else None
+        self.norm_ff = build_part(spec.norm_ff, rt) if spec.feed_forward is not None else None
+        self.share = None
+
+    def param_decls(self):
+        d = PreNormBlock.param_decls(self)
+        if self.spec.shift is not None:
+            d.append(ParamDecl(self.spec.shift, (self.spec.norm_mix.dim,), init="fraction", keep_float32=True))
+        return d
+
+    def bind(self, tensors):
+        if self.spec.shift is not None:
+            self.share = tensors.pop(self.spec.shift).to(torch.float32).contiguous()
+        PreNormBlock.bind(self, tensors)
+
+    def cache_requests(self):
+        r = list(self.mixer.cache_requests())
+        if self.spec.shift is not None:
+            r.append(StateRequest((self.spec.norm_mix.dim,), torch.float32))
+        return r
+
+    def forward(self, ctx, h, pending, views, writes=True, a=None):
+        dtype = self.rt.dtype
+        delta, norm = (pending.delta, norm_args(pending.norm)) if isinstance(pending, NormedDelta) else (pending, None)
+        a = torch.empty(h.shape, dtype=dtype, device=h.device)
+        save = None
+        seqs = ctx.sequence_rows()
+        if self.share is None:
+            api.sublayer_add(h, delta, norm, a, h_out=h if delta is not None else None)
+        else:
+            if not writes:
+                raise ValueError("a layer that reads the stream of the token before cannot run on another layer's cache entry")
+            *views, shift = views
+            save = shift.state
+            x = h if delta is None else torch.empty_like(h)
+            api.sublayer_add_shift(h, delta, norm, self.share, save, seqs, a, h_out=None if delta is None else x)
+            ctx.stream, h = x, x
+        d = self.mixer.forward(ctx, views, a, writes)
+        if self.feed_forward is None:
+            if save is not None:
+                cu_q, pos0, n_seq = ctx.sequences()
+                api.stream_save(h, save, cu_q, pos0, ctx.seq_slot, n_seq)
+            return NormedDelta(d, self.norm_mix)
+        # the state moves on here: every row of the step has read the old one by now, and h is what the mixer has read
+        a = torch.empty(h.shape, dtype=dtype, device=h.device)
+        api.sublayer_add(h, d, norm_args(self.norm_mix), a, h_out=h, save=save, seqs=seqs)
+        return NormedDelta(self.feed_forward.forward(ctx, a), self.norm_ff)
+
+
+register_part(OutputNormLayerSpec, OutputNormBlock)

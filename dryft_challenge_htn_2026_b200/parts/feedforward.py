@@ -42,33 +42,38 @@ register_part(GatedMLPSpec, GatedMLP)
 
 
 class DenseMLP(Part):
-    """down(act(up(x))) with the xIELU activation: act(z) = ap z^2 + z/2 for z > 0 and
+    """down(act(up(x))) with the squared ReLU, max(z, 0)^2, or the xIELU activation: act(z) = ap z^2 + z/2 for z > 0 and
     an (e^z - 1 - z) + z/2 otherwise, ap = softplus(p), an = 1/2 + softplus(q) from the two learned
     numbers of ``act`` (worked out once, in float64, when the tensors are bound). The activation sits in
     the epilogue of the up projection (every product kernel of the library has it as a mode)."""
 
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
-        if spec.activation != "xielu":
-            raise ValueError(f"activation {spec.activation!r} is not implemented (xielu only)")
+        if spec.activation not in ("xielu", "relu2"):
+            raise ValueError(f"activation {spec.activation!r} is not implemented (xielu, relu2)")
 
     def param_decls(self):
         s = self.spec
-        return [ParamDecl("up", (s.intermediate_size, s.hidden_size)), ParamDecl("down", (s.hidden_size, s.intermediate_size)),
-                ParamDecl("act", (2,), init="unit", keep_float32=True)]
+        d = [ParamDecl("up", (s.intermediate_size, s.hidden_size)), ParamDecl("down", (s.hidden_size, s.intermediate_size))]
+        if s.activation == "xielu":
+            d.append(ParamDecl("act", (2,), init="unit", keep_float32=True))
+        return d
 
     def bind(self, tensors):
         self.w_up = tensors.pop("up").contiguous()
         self.w_down = tensors.pop("down").contiguous()
+        if self.spec.activation == "relu2":
+            self.act = api.RELU2
+            return
         p, q = (float(x) for x in tensors.pop("act").to(torch.float64).cpu())
         softplus = lambda x: max(x, 0.0) + math.log1p(math.exp(-abs(x)))
-        self.alpha_pos, self.alpha_neg = softplus(p), 0.5 + softplus(q)
+        self.act = self.alpha_pos, self.alpha_neg = softplus(p), 0.5 + softplus(q)
 
     def step_weights(self):
         return [self.w_up, self.w_down]
 
     def forward(self, ctx, a):
-        z = linear(a, self.w_up, XIELU, act=(self.alpha_pos, self.alpha_neg))
+        z = linear(a, self.w_up, XIELU, act=self.act)
         return linear(z, self.w_down, allow_partial=True)
 
 

@@ -8,7 +8,8 @@ q_h . [c | k_rot] against the cached row itself -> attention with all heads on t
 attention's kernels: float32-arithmetic, mma.sync prompts, single tokens; rows wider than 256 on the kernel for rows that
 are key and value at once), whose values are the latents -> per head
 W_uv times the latent output -> output projection. Nothing per head is ever cached or recomputed for old tokens, so
-a step costs the same however a prompt is cut.
+a step costs the same however a prompt is cut. Without a query latent the queries come straight out of the first product;
+without rotated parts the cached row is the latent alone; a sink per head may join the softmax's denominator.
 """
 import torch
 
@@ -36,33 +37,51 @@ class LatentAttention(Part):
             raise ValueError(f"a rotation over {self.position.spec.dim} coordinates of a rotated part of {s.rot_dim}")
         self.lat = s.kv_rank + s.rot_dim                     # what a token holds in the cache: the key row
         self.n_q = s.num_heads * (s.head_dim + s.rot_dim)
-        self.n_down = s.q_rank + s.kv_rank + s.rot_dim
+        # the first product: [dq; dkv] with a query latent, [q; dkv] without one (filled up with zero rows to whole 16 bytes)
+        self.n_down = (s.q_rank or self.n_q) + s.kv_rank + s.rot_dim
+        self.n_fill = 0 if s.q_rank else -self.n_down % 8
         self.n_mid = s.num_heads * s.v_head_dim
         # the attention itself: every query head on the one cached head, keys [c | k_rot], values c
         self.core = MaskedAttention(MaskedAttentionSpec(
             hidden_size=s.hidden_size, num_heads=s.num_heads, num_kv_heads=1, head_dim=self.lat, v_head_dim=s.kv_rank,
-            scale=s.scale, chunk=s.chunk, window=s.window, values_in_keys=True), rt)
+            scale=s.scale, chunk=s.chunk, window=s.window, values_in_keys=True, sink=s.sink), rt)
         self.max_positions = 0
 
     def param_decls(self):
         s = self.spec
-        return [ParamDecl("dq", (s.q_rank, s.hidden_size)), ParamDecl("dq.norm", (s.q_rank,), init="norm", keep_float32=True),
-                ParamDecl("uq", (self.n_q, s.q_rank)), ParamDecl("dkv", (s.kv_rank + s.rot_dim, s.hidden_size)),
+        if s.q_rank:
+            q = [ParamDecl("dq", (s.q_rank, s.hidden_size)), ParamDecl("dq.norm", (s.q_rank,), init="norm", keep_float32=True),
+                 ParamDecl("uq", (self.n_q, s.q_rank))]
+        else:
+            q = [ParamDecl("q", (self.n_q, s.hidden_size))]
+        if s.sink:
+            q.append(ParamDecl("sink", (s.num_heads,), init="unit", keep_float32=True))
+        return q + [
+                ParamDecl("dkv", (s.kv_rank + s.rot_dim, s.hidden_size)),
                 ParamDecl("dkv.norm", (s.kv_rank,), init="norm", keep_float32=True),
                 ParamDecl("uk", (s.num_heads * s.head_dim, s.kv_rank)), ParamDecl("uv", (s.num_heads * s.v_head_dim, s.kv_rank)),
                 ParamDecl("o", (s.hidden_size, self.n_mid))]
 
     def bind(self, tensors):
-        self.w_down = torch.cat([tensors.pop("dq"), tensors.pop("dkv")], 0).contiguous()
-        self.q_norm_w = tensors.pop("dq.norm").to(torch.float32).contiguous()
+        if self.spec.sink:
+            self.core.sink = tensors.pop("sink").to(torch.float32).contiguous()
+        if self.spec.q_rank:
+            first = [tensors.pop("dq"), tensors.pop("dkv")]
+            self.q_norm_w = tensors.pop("dq.norm").to(torch.float32).contiguous()
+            self.w_uq = tensors.pop("uq").contiguous()
+        else:
+            first = [tensors.pop("q"), tensors.pop("dkv")]
+            if self.n_fill:
+                first.append(torch.zeros((self.n_fill, self.spec.hidden_size), dtype=first[0].dtype, device=first[0].device))
+            self.q_norm_w = self.w_uq = None
+        self.w_down = torch.cat(first, 0).contiguous()
         self.kv_norm_w = tensors.pop("dkv.norm").to(torch.float32).contiguous()
-        self.w_uq = tensors.pop("uq").contiguous()
         self.w_uk = tensors.pop("uk").contiguous()
         self.w_uv = tensors.pop("uv").contiguous()
         self.w_o = tensors.pop("o").contiguous()
 
     def step_weights(self):
-        return [self.w_down, self.w_uq, self.w_uk, self.w_uv, self.w_o]
+        return [w for w in (self.w_down, self.w_uq, self.w_uk, self.w_uv, self.w_o) if w is not None]
 
     def step_plans(self):
         return self.core.step_plans()
@@ -90,9 +109,10 @@ class LatentAttention(Part):
         out = torch.empty((T, H * self.lat), dtype=self.rt.dtype, device=self.rt.device)
         batched = self.rt.dtype == torch.bfloat16 and T > HEAD_PRODUCT_ROWS
         if batched:      # [H, T, D] x [H, D, L] -> the plain parts of out, seen as [H, T, L]
-            torch.bmm(q.view(T, H, D + R)[:, :, :D].transpose(0, 1), self.w_uk.view(H, D, L),
+            torch.bmm(q.unflatten(1, (H, D + R))[:, :, :D].transpose(0, 1), self.w_uk.view(H, D, L),
                       out=out.view(T, H, self.lat)[:, :, :L].transpose(0, 1))
-        api.latent_query(q, self.w_uk, out, cos, sin, rot, ctx.row_pos, H, D, R, L, plain=not batched)
+        if not batched or R:
+            api.latent_query(q, self.w_uk, out, cos, sin, rot, ctx.row_pos, H, D, R, L, plain=not batched)
         return out
 
     def values(self, o_lat):
@@ -111,12 +131,16 @@ class LatentAttention(Part):
         s, kv = self.spec, views[0]
         dtype, dev = self.rt.dtype, self.rt.device
         down = linear(a, self.w_down)
-        cq = torch.empty((ctx.n_tok, s.q_rank), dtype=dtype, device=dev)
         cos, sin, rot = self._tables(ctx)
-        api.latent_norm_rope_write(down, cq, self.q_norm_w, self.kv_norm_w, s.norm_eps, cos, sin, rot, ctx.row_pos,
-                                   ctx.row_seq, s.q_rank, s.kv_rank, s.rot_dim, kv.k if writes else None,
-                                   kv.v if writes else None, ctx.tables[kv.group] if writes else None)
-        q = self.queries(ctx, linear(cq, self.w_uq))
+        if s.q_rank:
+            cq, rows = torch.empty((ctx.n_tok, s.q_rank), dtype=dtype, device=dev), down
+        else:
+            cq, rows = None, down[:, self.n_q:self.n_down]
+        if s.q_rank or writes:
+            api.latent_norm_rope_write(rows, cq, self.q_norm_w, self.kv_norm_w, s.norm_eps, cos, sin, rot, ctx.row_pos,
+                                       ctx.row_seq, s.q_rank or 0, s.kv_rank, s.rot_dim, kv.k if writes else None,
+                                       kv.v if writes else None, ctx.tables[kv.group] if writes else None)
+        q = self.queries(ctx, linear(cq, self.w_uq) if s.q_rank else down[:, :self.n_q])
         o_lat = torch.empty((ctx.n_tok, s.num_heads * s.kv_rank), dtype=dtype, device=dev)
         self.core.attend(ctx, kv, q, None, None, None, o_lat, 1.0, writes=False)
         return linear(self.values(o_lat), self.w_o, allow_partial=True)

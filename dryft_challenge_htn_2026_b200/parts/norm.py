@@ -1,22 +1,25 @@
 """RMSNorm (reference: engine/engine.py:107-110, engine/fused.py:152-172)."""
 import torch
 
-from ..config.specs import GroupRMSNormSpec, OnePlusRMSNormSpec, RMSNormSpec, ScalarRMSNormSpec
+from ..config.specs import GroupRMSNormSpec, LayerNormSpec, OnePlusRMSNormSpec, RMSNormSpec, ScalarRMSNormSpec
 from ..csrc import api
 from .base import ParamDecl, Part, register_part
 
 
 class NormedDelta:
     """A sublayer's output that still has to go through a norm of its own before it joins the residual stream:
-    ``delta`` (a tensor or a ``csrc.api.Partial``) and ``norm`` (an ``RMSNorm`` part). The norm that follows the sum
-    takes it as its ``delta`` and does both in one kernel."""
+    ``delta`` (a tensor, a ``csrc.api.Partial`` or a ``csrc.api.NormedSum``) and ``norm`` (an ``RMSNorm`` or ``LayerNorm``
+    part). What follows the sum (a norm, or the next block's own sum) takes it as its ``delta`` and does both in one kernel."""
 
     def __init__(self, delta, norm):
         self.delta, self.norm = delta, norm
 
     def to_float32(self):
         """What joins the stream, worked out plainly (for dumps of the stream between layers)."""
-        d = self.delta.ws.sum(0) if isinstance(self.delta, api.Partial) else self.delta.to(torch.float32)
+        d = self.delta.to_float32() if isinstance(self.delta, api.NormedSum) else \
+            self.delta.ws.sum(0) if isinstance(self.delta, api.Partial) else self.delta.to(torch.float32)
+        if isinstance(self.norm, LayerNorm):
+            d = d - d.mean(-1, keepdim=True)
         return d * torch.rsqrt((d * d).mean(-1, keepdim=True) + self.norm.spec.eps) * self.norm.weight
 
 
@@ -105,3 +108,42 @@ class GroupRMSNorm(Part):
 
 
 register_part(GroupRMSNormSpec, GroupRMSNorm)
+
+
+class LayerNorm(Part):
+    """Layer norm with a weight and no bias, y = w * (x - mean) / sqrt(variance + eps), the variance the mean of the squared
+    deviations (taken of the deviations themselves, not of the squares). Statistics in float32, weight held in float32. It
+    runs in the kernel that adds a sublayer's output to the stream: as the norm of that output (``OutputNormBlock``) and as
+    the norm behind the sum (``add_forward``)."""
+    takes_partial = True
+    takes_normed = True      # add_forward also takes a sublayer's output that has a norm of its own (NormedDelta)
+
+    def param_decls(self):
+        return [ParamDecl(self.spec.tensor, (self.spec.dim,), init="norm", keep_float32=True)]
+
+    def bind(self, tensors):
+        self.weight = tensors[self.spec.tensor].to(torch.float32).contiguous()
+
+    def args(self):
+        """(weight, eps, center) as ``csrc.api.sublayer_add`` takes a norm."""
+        return self.weight, self.spec.eps, True
+
+    def add_forward(self, h, delta, out, rows=None):
+        """h += delta, out = norm(h); with ``rows`` of those rows only, leaving h as it is."""
+        norm = None
+        if isinstance(delta, NormedDelta):
+            delta, norm = delta.delta, norm_args(delta.norm)
+        api.sublayer_add(h, delta, norm, out, h_out=h if rows is None else None, rows=rows, next_norm=self.args())
+        return out
+
+
+register_part(LayerNormSpec, LayerNorm)
+
+
+def norm_args(norm):
+    """(weight, eps, center) of a norm part, as ``csrc.api.sublayer_add`` takes it."""
+    if isinstance(norm, LayerNorm):
+        return norm.args()
+    if isinstance(norm, RMSNorm):
+        return norm.weight, norm.spec.eps, False
+    raise TypeError(f"{type(norm).__name__} cannot stand on a sublayer's output")

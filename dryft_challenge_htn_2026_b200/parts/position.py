@@ -8,6 +8,8 @@ for one that rewrites the q and k heads of the projection rows [tokens, (nh + 2 
 itself; the attention part then runs the fused kernel without rotation. ``apply`` runs before the
 cache write and cannot be combined with a per-head q/k norm (which would have to come first): the
 attention part refuses that pair."""
+import math
+
 import torch
 
 from ..config.specs import RotaryHalfSpec, RotaryPairsSpec, RotaryPartSpec, SinusoidSpec
@@ -51,6 +53,16 @@ class Sinusoid(Part):
 register_part(SinusoidSpec, Sinusoid)
 
 
+def stretched(freq, dim, base, factor, original, fast, slow):
+    """YaRN: pairs that turn often within ``original`` positions keep their frequency, those that turn seldom have it divided
+    by ``factor``, with a linear ramp between the pairs that turn ``fast`` and ``slow`` times. -> (frequencies, factor on
+    sine and cosine)"""
+    at = lambda turns: dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), dim - 1)
+    ramp = ((torch.arange(freq.numel(), dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 class RotaryPart(Part):
     """Angle tables of a rotation over the first ``dim`` coordinates of a head: frequencies base^(-2i/dim) made
     in float64 and rounded to float32 once, angle = float32(position) * frequency in float32, its cosine and
@@ -71,10 +83,14 @@ class RotaryPart(Part):
             n = max(n, 2 * self._n, 256)
             dim = self.spec.dim
             i = torch.arange(dim // 2, dtype=torch.float64)
-            freq = (float(self.spec.base) ** (-2.0 * i / dim)).to(torch.float32)
+            freq = float(self.spec.base) ** (-2.0 * i / dim)
+            amplitude = 1.0
+            if self.spec.scaling is not None:
+                freq, amplitude = stretched(freq, dim, float(self.spec.base), *self.spec.scaling)
+            freq = freq.to(torch.float32)
             ang = (torch.arange(n, dtype=torch.float32)[:, None] * freq[None, :]).to(torch.float64)
-            self._cos = ang.cos().to(torch.float32).to(self.rt.device).contiguous()
-            self._sin = ang.sin().to(torch.float32).to(self.rt.device).contiguous()
+            self._cos = (ang.cos() * amplitude).to(torch.float32).to(self.rt.device).contiguous()
+            self._sin = (ang.sin() * amplitude).to(torch.float32).to(self.rt.device).contiguous()
             self._n = n
         return self._cos, self._sin
 

@@ -20,14 +20,6 @@ from .base import ParamDecl, Part, register_part
 from .linear import linear
 
 
-def _sequences(ctx):
-    """(cu_q, seq_pos0, n_seq) as the recurrence kernels want them: one token a row in a decode step (padding rows carry
-    position -1), else the step's sequences."""
-    if ctx.is_decode:
-        return None, ctx.row_pos, ctx.n_tok
-    return ctx.cu_q, ctx.seq_pos0, ctx.n_seq
-
-
 class LowerBoundRecurrence(Part):
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
@@ -67,7 +59,7 @@ class LowerBoundRecurrence(Part):
         q, k, v, a = api.recurrence_operands(T, self.n_qk, self.n_mid, dev)
         api.hgrn2_prepare(proj[:, :self.n_in], self.f_bias, self.lower, q, k, a, v)
         o = torch.empty((T, self.n_mid), dtype=torch.float32, device=dev)
-        cu_q, pos0, n_seq = _sequences(ctx)
+        cu_q, pos0, n_seq = ctx.sequences()
         api.recurrence(q, k, a, v, o, views[0].state, cu_q, pos0, ctx.seq_slot, n_seq, s.num_heads, s.head_dim, s.v_head_dim)
         api.norm_gate(o, self.norm_weight, s.norm_eps, None, scale, mid, group=s.v_head_dim)
 
@@ -136,7 +128,7 @@ class StateSpace(Part):
         conv_state = views[1].state if s.conv_taps > 1 else None
         # the recurrence's operands head by head: q = C and k = dt B of the head's group, the head's decay on every channel
         q, k, x, a = api.recurrence_operands(T, s.num_heads * s.state_dim, inner, dev)
-        cu_q, pos0, n_seq = _sequences(ctx)
+        cu_q, pos0, n_seq = ctx.sequences()
         api.ssd_prepare(xbc, dt, conv_state, self.w_conv, self.conv_bias, s.conv_taps, self.dt_bias, self.a_log, ctx.row_pos,
                         ctx.row_seq, pos0, ctx.seq_slot, s.groups, q, k, a, x)
         if s.conv_taps > 1:
