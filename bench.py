@@ -954,8 +954,188 @@ def nevotar_kernel_times(torch, dk, pk, cfg_d, p_cfg):
     return out
 
 
+def fukatar_config(width, heads, kv_heads, ff_qwen, layers, vocab):
+    """A Fukatar model of Qwen3's width, layer count and parameters in the feed-forward: a layer of two mixers side by side
+    (attention of half Qwen3's head counts, half the head rotated by pairs, scores capped, beside the gated delta rule with as
+    many heads of 128 x 128 on half as many key heads, 4 taps), a layer of Qwen3's head counts with whole-projection norms,
+    stretched positions, capped scores, turning values and a gate per head, and two layers of attention through latents of 512
+    with plain key and value heads of 128 and a sink; a squared-ReLU feed-forward as large as Qwen3's gated one; rows of token
+    pairs and capped logits."""
+    hd, h2, g2 = 128, heads // 2, max(1, kv_heads // 2)
+    mlp = {"kind": "dense", "ff": 3 * ff_qwen // 2 // 64 * 64}
+    par = {"type": "parallel",
+           "mixer": {"left": {"heads": h2, "kv_heads": g2, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 50.0, "rot": {"dims": hd // 2, "base": 1e4}},
+                     "right": {"heads": h2, "kv_heads": h2 // 2, "dim": hd, "vdim": hd, "conv": 4}}, "mlp": mlp}
+    att = {"type": "attention",
+           "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0,
+                     "rot": {"dims": hd, "base": 1e6, "scaling": {"factor": 4.0, "original": 32768, "fast": 32.0, "slow": 1.0}}}, "mlp": mlp}
+    lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": hd, "vdim": hd, "kv_rank": 512, "scale": hd ** -0.5}, "mlp": mlp}
+    return dict(architecture="Fukatar", vocab=vocab, width=width, norm={"eps": 1e-6}, logit_softcap=30.0,
+                embedding={"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+                layers=[(par, att, lat, lat)[i % 4] for i in range(layers)])
+
+
+def fukatar_kernel_times(torch, dk, pk, cfg_d, p_cfg):
+    """The design's steps alone (the parts of a model of ``cfg_d``, so each step runs whichever kernel the part picks), with
+    gated linear attention of the Pibulix model ``p_cfg`` beside the delta rule: CUDA events around one step, L2 flushed
+    before each (a 256 MB write), median of 5 after 2 untimed. Prompts' attention and products against the bfloat16 peak,
+    everything else against the copy peak by the bytes the step must move."""
+    from dryft_challenge_htn_2026_b200.cache import Cache, StateRequest
+    from dryft_challenge_htn_2026_b200.csrc import api
+    from dryft_challenge_htn_2026_b200.engine.batch import build_context
+    from dryft_challenge_htn_2026_b200.parts import Runtime, build_part
+    from dryft_challenge_htn_2026_b200.parts.linear import XIELU, linear
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
+
+    def timed(fn):
+        ts = []
+        for i in range(7):
+            flush.fill_(float(i))
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        return statistics.median(ts[2:]) * 1e3        # microseconds
+
+    def flops_rec(us, flops):
+        return {"us": round(us, 1), "tflops": round(flops / us / 1e6, 1), "frac_bf16": round(flops / us / 1e6 / pk["bf16_tflops"], 4)}
+
+    def bytes_rec(us, moved):
+        return {"us": round(us, 1), "gbs": round(moved / us / 1e3, 1), "frac_hbm": round(moved / us / 1e3 / pk["hbm_gbs"], 4)}
+
+    rt = Runtime(dev, bf)
+    g = torch.Generator(device=dev).manual_seed(1)
+    spec, pspec = dk.config_from_dict(cfg_d).to_spec(), dk.config_from_dict(p_cfg).to_spec()
+    W = spec.hidden_size
+
+    def bound(part_spec):
+        part = build_part(part_spec, rt)
+        part.bind({d.name: (torch.rand(d.shape, generator=g, device=dev) * 0.5 if d.init == "fraction" else
+                            torch.randn(d.shape, generator=g, device=dev) * (0.2 if d.init in ("wide", "taps") else 0.02) + (1.0 if d.init == "norm" else 0.0)).to(
+            torch.float32 if d.keep_float32 else bf) for d in part.param_decls()})
+        part.prepare(16384)
+        return part
+
+    par, att, lat = (bound(spec.layers[i].mixer) for i in range(3))
+    left, delta = par.branches[0][1], par.branches[1][1]
+    ff, p_gla = bound(spec.layers[0].feed_forward), bound(pspec.layers[1].mixer)
+    ls, ds = lat.spec, delta.spec
+    w = torch.ones(W, device=dev)
+    share = torch.full((W,), 0.3, device=dev)
+    out = {}
+
+    def fill(cache, n):
+        for e in range(n):
+            for v in cache.views(e):
+                if hasattr(v, "k"):
+                    v.k.normal_()
+                    if v.v is not None:
+                        v.v.normal_()
+
+    def steps(ctx, cache, rows, tag, pairs, keys):
+        """``pairs``: (query, key) pairs in sight in a prompt (0: single tokens that read ``keys`` keys each)."""
+        ctx.carry = {}
+        for name, part, views in (("turning_values", att, cache.views(1)), ("pairs", left, cache.views(0)[:1])):
+            s = part.spec
+            proj = (torch.randn(rows, part.n_in, device=dev) * 0.5).to(bf)
+            mid = torch.empty(rows, part.n_mid, dtype=bf, device=dev)
+            q = part.rotated_queries(ctx, views, proj)
+            us = timed(lambda: part.rotated_queries(ctx, views, proj))
+            out[f"rows_{name}_{tag}"] = bytes_rec(us, rows * part.n_qkv * 2 * 2)
+            us = timed(lambda: part.attend(ctx, views[0], q, None, None, None, mid, 1.0, writes=False))
+            out[f"attention_{name}_{tag}"] = flops_rec(us, 4 * s.num_heads * s.head_dim * pairs) if pairs else \
+                dict(bytes_rec(us, rows * s.num_kv_heads * keys * 2 * s.head_dim * 2), keys=keys)
+            if part.behind:
+                gate, rot = proj[:, part.n_qkv:part.n_qkv + part.n_gate], part._rotation(ctx, part.value_position)
+                us = timed(lambda: api.turn_back_gate(mid, mid, gate, rot, 1.0, ctx.row_pos, s.num_heads, s.v_head_dim))
+                out[f"turn_back_gate_{tag}"] = bytes_rec(us, rows * part.n_mid * 2 * 2)
+        kv, H, D, L, Dv = cache.views(2)[0], ls.num_heads, ls.head_dim, ls.kv_rank, ls.v_head_dim
+        down = torch.randn(rows, lat.n_down + lat.n_fill, device=dev).to(bf)
+        table = ctx.tables[kv.group]
+        us = timed(lambda: api.latent_norm_rope_write(down[:, lat.n_q:lat.n_down], None, None, lat.kv_norm_w, ls.norm_eps, None, None, 0, ctx.row_pos,
+                                                      ctx.row_seq, 0, L, 0, kv.k, None, table))
+        out[f"latent_norm_cache_write_{tag}"] = bytes_rec(us, rows * L * 2 * 2)
+        ql = lat.queries(ctx, down[:, :lat.n_q])
+        us = timed(lambda: lat.queries(ctx, down[:, :lat.n_q]))
+        out[f"latent_query_heads_{tag}"] = flops_rec(us, 2 * rows * H * D * L) if pairs else bytes_rec(us, H * D * L * 2 + rows * (lat.n_q + H * L) * 2)
+        o_lat = torch.empty(rows, H * L, dtype=bf, device=dev)
+        us = timed(lambda: lat.core.attend(ctx, kv, ql, None, None, None, o_lat, 1.0, writes=False))
+        out[f"latent_attention_{tag}"] = flops_rec(us, 4 * H * L * pairs) if pairs else dict(bytes_rec(us, rows * keys * L * 2), keys=keys)
+        us = timed(lambda: lat.values(o_lat))
+        out[f"latent_value_heads_{tag}"] = flops_rec(us, 2 * rows * H * Dv * L) if pairs else bytes_rec(us, H * Dv * L * 2 + rows * (H * L + lat.n_mid) * 2)
+        del ql, o_lat, down
+        # the recurrences: what a prompt must move (operands in float32 in, outputs out), what a single token must (the state, twice)
+        proj = (torch.randn(rows, delta.n_in, device=dev) * 0.5).to(bf)
+        mid = torch.empty(rows, delta.n_mid, dtype=bf, device=dev)
+        views = cache.views(0)[1:3]
+        state_bytes = rows * ds.num_heads * ds.head_dim * ds.v_head_dim * 4 * 2
+        moved = rows * (2 * ds.num_kv_heads * ds.head_dim + 2 * ds.num_heads * ds.v_head_dim) * 4
+        us = timed(lambda: delta.mix(ctx, views, proj, mid, 1.0))
+        out[f"delta_rule_mixer_{tag}"] = bytes_rec(us, moved if pairs else state_bytes)
+        cu_q, pos0, n_seq = ctx.sequences()
+        sizes = (ds.num_heads, ds.num_kv_heads, ds.head_dim, ds.v_head_dim)
+        qkv, scal = api.delta_operands(rows, *sizes, dev)
+        c = delta.n_conv + delta.n_mid
+        us = timed(lambda: api.delta_prepare(proj[:, :delta.n_conv], proj[:, c + ds.num_heads:c + 2 * ds.num_heads], proj[:, c:c + ds.num_heads], views[1].state,
+                                             delta.w_conv, ds.conv_taps, delta.a_log, delta.dt_bias, ds.unit_eps, ctx.row_pos, ctx.row_seq, pos0,
+                                             ctx.seq_slot, qkv, scal, *sizes))
+        out[f"delta_operands_{tag}"] = bytes_rec(us, rows * delta.n_conv * (2 + 4))
+        o = torch.empty(rows, delta.n_mid, dtype=torch.float32, device=dev)
+        us = timed(lambda: api.delta_rule(qkv, scal, o, views[0].state, cu_q, pos0, ctx.seq_slot, n_seq, *sizes))
+        out[f"delta_recurrence_{tag}"] = bytes_rec(us, moved if pairs else state_bytes)
+        gs = p_gla.spec
+        pg, mg = torch.randn(rows, p_gla.n_in, device=dev).to(bf), torch.empty(rows, p_gla.n_mid, dtype=bf, device=dev)
+        us = timed(lambda: p_gla.mix(ctx, cache.views(3), pg, mg, 1.0))
+        out[f"pibulix_gated_linear_attention_{tag}"] = bytes_rec(us, rows * gs.num_heads * (3 * gs.head_dim + 2 * gs.v_head_dim) * 4 if pairs else
+                                                                 rows * gs.num_heads * gs.head_dim * gs.v_head_dim * 4 * 2)
+        # the stream
+        h, x, a = torch.randn(rows, W, device=dev), torch.empty(rows, W, device=dev), torch.randn(rows, W, device=dev).to(bf)
+        b, o = torch.randn(rows, W, device=dev).to(bf), torch.empty(rows, W, dtype=bf, device=dev)
+        shift, seqs, norm = cache.views(2)[1].state, ctx.sequence_rows(), (w, 1e-6, True)
+        us = timed(lambda: api.sublayer_add_shift(h, a, norm, share, shift, seqs, o, h_out=x))
+        out[f"output_norm_sum_shift_{tag}"] = bytes_rec(us, rows * W * (4 + 2 + 4 + 2))
+        us = timed(lambda: api.sublayer_add(h, a, norm, o, h_out=h, save=shift, seqs=seqs))
+        out[f"output_norm_sum_{tag}"] = bytes_rec(us, rows * W * (4 + 2 + 4 + 2))
+        two = api.NormedSum([a, b], [w, w], 1e-6, 0.5)
+        us = timed(lambda: api.sublayer_add(h, two, norm, o, h_out=h, save=shift, seqs=seqs))
+        out[f"two_output_norms_sum_{tag}"] = bytes_rec(us, rows * W * (4 + 4 + 4 + 2))
+        us = timed(lambda: api.normed_add_rmsnorm(h, a, w, 1e-6, w, 1e-6, o))
+        out[f"venidra_output_norm_sum_norm_{tag}"] = bytes_rec(us, rows * W * (4 + 2 + 4 + 2))
+        us = timed(lambda: linear(a, ff.w_up, XIELU, act=ff.act))
+        out[f"squared_relu_product_{tag}"] = flops_rec(us, 2 * rows * ff.w_up.numel()) if pairs else bytes_rec(us, ff.w_up.numel() * 2)
+        us = timed(lambda: linear(a, ff.w_up))
+        out[f"plain_product_{tag}"] = flops_rec(us, 2 * rows * ff.w_up.numel()) if pairs else bytes_rec(us, ff.w_up.numel() * 2)
+
+    entries = [par.cache_requests(), att.cache_requests(), lat.cache_requests() + [StateRequest((W,), torch.float32)], p_gla.cache_requests()]
+    plans = list({p.key: p for part in (par, att, lat) for p in part.step_plans()}.values())
+    for tokens in (2048, 8192):
+        cache = Cache(entries, tokens + 64, 2, dev)
+        slot = cache.begin()
+        ctx = build_context(cache, [(slot, [0] * tokens, [])], dev, plans=plans)
+        fill(cache, 4)
+        steps(ctx, cache, tokens, str(tokens), tokens * (tokens + 1) // 2, 0)
+        cache.end(slot)
+        del cache
+    for batch in (8, 64):
+        context = 3000
+        cache = Cache(entries, batch * (context + 64), batch, dev)
+        slots = [cache.begin() for _ in range(batch)]
+        for sl in slots:
+            cache.reserve(sl, context + 1)
+            cache.length[sl] = context
+        ctx = build_context(cache, [(sl, [0], []) for sl in slots], dev, plans=plans)
+        fill(cache, 4)
+        steps(ctx, cache, batch, f"decode_b{batch}", 0, context + 1)
+        del cache
+    torch.cuda.empty_cache()
+    return out
+
+
 def run_design(args):
-    """``--design nilivik`` / ``--design pibulix`` / ``--design venidra`` / ``--design nevotar``: prefill and decode of that decoder at Qwen3 layer sizes (random weights,
+    """``--design nilivik`` / ``--design pibulix`` / ``--design venidra`` / ``--design nevotar`` / ``--design fukatar``: prefill and decode of that decoder at Qwen3 layer sizes (random weights,
     ``--layers`` layers, default 4) beside Qwen3 itself at the same width, layer count and parameters a
     layer, and the design's mixer kernels alone beside Qwen3's attention kernels. One JSON line."""
     import torch
@@ -968,12 +1148,19 @@ def run_design(args):
     layers = args.layers or 4
     chunk = 2048
     vocab = 32768
-    out = {"design": args.design, "beside": "Pibulix" if args.design == "nevotar" else "Qwen3ForCausalLM", "layers": layers, "chunk": chunk, "vocab": vocab, "dtype": "bf16",
+    out = {"design": args.design, "beside": {"nevotar": "Pibulix", "fukatar": "Venidra"}.get(args.design, "Qwen3ForCausalLM"), "layers": layers, "chunk": chunk, "vocab": vocab, "dtype": "bf16",
            "data": "synthetic: random weights, uniform random token ids", "peaks": pk, "sizes": {}}
     for size in args.design_sizes.split(","):
         q = dict(SIZES[size]["config"], num_hidden_layers=layers, vocab_size=vocab, tie_word_embeddings=True)
         beside = ("qwen3", q)
-        if args.design == "nevotar":
+        sizes = (q["hidden_size"], q["num_attention_heads"], q["num_key_value_heads"], q["intermediate_size"], layers, vocab)
+        if args.design == "fukatar":
+            n = fukatar_config(*sizes)
+            beside = ("venidra", venidra_config(*sizes))
+            rec = {"width": q["hidden_size"], "ff": n["layers"][0]["mlp"]["ff"], "kv_rank": 512,
+                   "beside": "Venidra of the same width, layer count and feed-forward parameters (the closest of the library's designs: "
+                             "attention with a rotation and a unit norm in turn with attention through latents, norms on the outputs)"}
+        elif args.design == "nevotar":
             n = nevotar_config(q["hidden_size"], q["num_attention_heads"], q["num_key_value_heads"], q["intermediate_size"], layers, vocab)
             beside = ("pibulix", pibulix_config(q["hidden_size"], q["num_attention_heads"], q["num_key_value_heads"], q["intermediate_size"],
                                                 layers, vocab, PIBULIX_WINDOW))
@@ -1005,7 +1192,10 @@ def run_design(args):
             rec[name] = r
             del model
             torch.cuda.empty_cache()
-        if args.design == "nevotar":
+        if args.design == "fukatar":
+            rec["kernels"] = fukatar_kernel_times(torch, dk, pk, n, pibulix_config(*sizes, PIBULIX_WINDOW))
+            rec["venidra_kernels"] = venidra_kernel_times(torch, dk, pk, beside[1], q["num_attention_heads"], q["num_key_value_heads"])
+        elif args.design == "nevotar":
             rec["kernels"] = nevotar_kernel_times(torch, dk, pk, n, beside[1])
         elif args.design == "venidra":
             rec["kernels"] = venidra_kernel_times(torch, dk, pk, n, q["num_attention_heads"], q["num_key_value_heads"])
@@ -1220,9 +1410,9 @@ def main():
     ap.add_argument("--prefill-only", action="store_true", help="only the 2,048-token prefill (for profiling its kernels)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="with --prefill-only: a prompt of another length")
     ap.add_argument("--pdl", type=int, default=1, help="programmatic dependent launch on (1) or off (0)")
-    ap.add_argument("--design", default=None, choices=["nilivik", "pibulix", "venidra", "nevotar"],
+    ap.add_argument("--design", default=None, choices=["nilivik", "pibulix", "venidra", "nevotar", "fukatar"],
                     help="instead of the default workload: prefill and decode of this design at Qwen3 layer sizes beside Qwen3 "
-                         "itself at equal size (nevotar: beside Pibulix, the closest of the library's designs), and its mixer "
+                         "itself at equal size (nevotar: beside Pibulix, fukatar: beside Venidra, the closest of the library's designs), and its mixer "
                          "kernels alone (one JSON line of its own)")
     ap.add_argument("--design-sizes", default="4b,8b", help="with --design: which of the layer sizes")
     args = ap.parse_args()

@@ -1,0 +1,66 @@
+"""A mixer part with random tensors, and the part over one sequence cut into steps of given lengths beside another sequence."""
+import torch
+
+from dryft_challenge_htn_2026_b200.cache import Cache
+from dryft_challenge_htn_2026_b200.csrc import api
+from dryft_challenge_htn_2026_b200.engine.batch import build_context
+from dryft_challenge_htn_2026_b200.parts import Runtime, build_part
+
+DEV = torch.device("cuda")
+
+
+def tol(dtype, ref):
+    return (2e-4 if dtype in (torch.float32, "float32") else 6e-2) * max(1.0, float(ref.abs().max()))
+
+
+def rnd(*shape, seed=0, scale=1.0):
+    return torch.randn(*shape, generator=torch.Generator().manual_seed(seed), dtype=torch.float64) * scale
+
+
+def close(got, ref, dtype, what="", slack=0.5):
+    err = float((got.double().cpu() - ref.double()).abs().max())
+    assert err <= tol(dtype, ref) * slack, f"{what}: max error {err} > {tol(dtype, ref) * slack}"
+
+
+def dev(x, dtype):
+    return x.to(dtype).to(DEV)
+
+
+def bound_part(spec, dtype, seed=0, scale=0.3, **given):
+    """-> (part, its tensors as float64 after the rounding the part's type does to them); ``given``: tensors by name."""
+    part = build_part(spec, Runtime(DEV, dtype))
+    p = {}
+    for i, d in enumerate(part.param_decls()):
+        x = rnd(*d.shape, seed=seed + 7 * i + 1)
+        x = {"norm": 1 + 0.2 * x, "fraction": torch.sigmoid(x), "taps": 0.6 * x, "unit": x}.get(d.init, scale * x)
+        if d.name in given:
+            x = given[d.name].double()
+        p[d.name] = x.to(torch.float32 if d.keep_float32 else dtype).double()
+    part.bind({d.name: dev(p[d.name], torch.float32 if d.keep_float32 else dtype) for d in part.param_decls()})
+    return part, p
+
+
+def whole(out):
+    """A part's output as float64 on the host, whatever form it comes in."""
+    if isinstance(out, api.NormedSum):
+        return out.to_float32().double().cpu()
+    return (out.ws.sum(0) if isinstance(out, api.Partial) else out).double().cpu()
+
+
+def run_cut(part, rows, lens, dtype):
+    """The part over one sequence of input rows cut into steps of ``lens``, a second sequence of other rows beside it in
+    every step (three tokens, or one when the step is a single token): -> the outputs of the first sequence's rows."""
+    cache = Cache([part.cache_requests()], 64 * 40, 4, DEV)
+    other, slot = cache.begin(), cache.begin()
+    part.prepare(sum(lens) + 8)
+    noise = rnd(4, rows.shape[1], seed=99)
+    got, t0 = [], 0
+    for n in lens:
+        m = 1 if n == 1 else 3
+        ctx = build_context(cache, [(other, [0] * m, []), (slot, [0] * n, [])], DEV, plans=part.step_plans())
+        ctx.carry = {}
+        a = torch.cat([dev(noise[:m], dtype), dev(rows[t0:t0 + n], dtype)], 0).contiguous()
+        got.append(whole(part.forward(ctx, cache.views(0), a))[m:])
+        cache.commit(other, m), cache.commit(slot, n)
+        t0 += n
+    return torch.cat(got, 0)
