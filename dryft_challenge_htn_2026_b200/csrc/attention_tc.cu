@@ -434,7 +434,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             const uint32_t t = step + i, b = t & 1, ph = (t >> 1) & 1;
             const int key0 = (i < cur.n_kept ? i : blk_lo + i - cur.n_kept) * BN;
 #if DK_MASKED
-            {   // this step's bias table, while S is still on its way (zeros without a bias)
+            if (b1 != 0.f || i < 2) {   // this step's bias table, while S is still on its way (without a bias two tables of zeros, once)
                 float* tw = bias_tab + (t & 1) * BIAS_TAB;
                 const int d_first = min_pos + (warp & 3) * 32 - key0 - (BN - 1);
                 for (int k = lane; k < BIAS_TAB; k += 32)
@@ -456,17 +456,42 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             // of the step sits at tab[lane + 63 - j] (distance = first distance of the warp in this step + that index)
             const float* tab = bias_tab + (t & 1) * BIAS_TAB + lane + (BN - 1);
             if (cap_l2 > 0.f) {
-                // capped scores: cap * tanh(score / cap), here times log2(e); tanh(y) = 1 - 2 / (e^(2y) + 1) from one
-                // exponential and one fast division (the hardware's own tanh is good to 11 bits only, which a cap of
-                // some tens of units turns into percents of a weight)
+                // capped scores: cap * tanh(score / cap), here times log2(e). Where all of the warp's scores are small
+                // against the cap, by the Taylor series of tanh (its next term is below 3e-8 at 0.4); else tanh(y) = 1 - 2 /
+                // (e^(2y) + 1) from one exponential and one fast division (the hardware's own tanh is good to 11 bits
+                // only, which a cap of some tens of units turns into percents of a weight)
+                float big4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                for (int j = 0; j < CPT; j++) {
-                    const float e = ex2(__uint_as_float(v[j]) * scale_over_cap * 2.8853900817779268f);
-                    v[j] = __float_as_uint(cap_l2 * (1.f - __fdividef(2.f, e + 1.f)));
+                for (int j = 0; j < CPT; j++) big4[j & 3] = fmaxf(big4[j & 3], fabsf(__uint_as_float(v[j])));
+                const float big = fmaxf(fmaxf(big4[0], big4[1]), fmaxf(big4[2], big4[3])) * fabsf(scale_over_cap);
+                if (__all_sync(0xffffffffu, big <= 0.4f)) {
+                    const float lead = cap_l2 * scale_over_cap, s2 = scale_over_cap * scale_over_cap;
+#pragma unroll
+                    for (int j = 0; j < CPT; j++) {
+                        const float x = __uint_as_float(v[j]), t2 = x * x * s2;
+                        float p = fmaf(t2, -1382.f / 155925.f, 62.f / 2835.f);
+                        p = fmaf(t2, p, -17.f / 315.f);
+                        p = fmaf(t2, p, 2.f / 15.f);
+                        p = fmaf(t2, p, -1.f / 3.f);
+                        v[j] = __float_as_uint(x * fmaf(t2 * lead, p, lead));
+                    }
+                } else {
+#pragma unroll
+                    for (int j = 0; j < CPT; j++) {
+                        const float e = ex2(__uint_as_float(v[j]) * scale_over_cap * 2.8853900817779268f);
+                        v[j] = __float_as_uint(cap_l2 * (1.f - __fdividef(2.f, e + 1.f)));
+                    }
                 }
             }
             const float sl = cap_l2 > 0.f ? 1.f : sl2;
-            if (open) {
+            if (open && b1 == 0.f) {
+#pragma unroll
+                for (int j = 0; j < CPT; j++) {
+                    const float x = __uint_as_float(v[j]) * sl;
+                    v[j] = __float_as_uint(x);
+                    mx4[j & 3] = fmaxf(mx4[j & 3], x);
+                }
+            } else if (open) {
 #pragma unroll
                 for (int j = 0; j < CPT; j++) {
                     const float x = fmaf(__uint_as_float(v[j]), sl, -tab[-j]);

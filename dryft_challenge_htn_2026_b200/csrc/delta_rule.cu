@@ -5,11 +5,11 @@
 //                      of q, k and v (its memory, the last taps - 1 projected rows, is a per-sequence state, read only
 //                      here), SiLU; q and k over sqrt(sum of squares + unit_eps) per head, q times D^(-1/2); g = exp(-exp(A)
 //                      softplus(a + dt)), beta = sigmoid(b); and k . q per key head (below).
-//   * delta_rule     : portions. One reduction over the state's rows a token: with a = S^T k and b = S^T q of the state as
-//                      the token finds it, u = beta (v - g a) and o = g b + (k . q) u. Eight lanes share a column of the
-//                      state, each with D / 8 of its rows in registers for the whole portion; the rows q, k, v of 16 tokens
-//                      at a time come through shared memory by cp.async, three chunks in turn.
-//   * delta_rule_step: one token a sequence: a block per (sequence, head, 32 columns) passes once over its part of the state.
+//   * delta_rule     : portions, four tokens a turn. Eight lanes share a column of the state, each with D / 8 of its rows in
+//                      registers for the whole portion; the rows q, k, v of 16 tokens at a time come through shared memory by
+//                      cp.async, three chunks in turn.
+//   * delta_rule_step: one token a sequence: a block per (sequence, head, 32 columns) passes once over its part of the state:
+//                      with a = S^T k and b = S^T q of the state as the token finds it, u = beta (v - g a), o = g b + (k . q) u.
 // Rows with position < 0 are padding: zeros out, states untouched.
 #include "common.cuh"
 
@@ -127,14 +127,36 @@ __device__ __forceinline__ void dr_cp(float* smem, const float* gmem, bool wide)
     else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(a), "l"(gmem) : "memory");
 }
 
+// The 16 sums a turn of four tokens needs over the lanes of a warp: halves are exchanged while more than one value is left,
+// then a plain sum; lane l ends with the sum of value l / 2.
+__device__ __forceinline__ float dr_fold16(float (&d)[16], int lane) {
+#pragma unroll
+    for (int n = 8; n >= 1; n >>= 1) {
+        const bool up = lane & (2 * n);
+#pragma unroll
+        for (int i = 0; i < n; i++) {
+            const float send = up ? d[i] : d[i + n], keep = up ? d[i + n] : d[i];
+            d[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2 * n);
+        }
+    }
+    return d[0] + __shfl_xor_sync(0xffffffffu, d[0], 1);
+}
+
 // grid (sequences, heads, ceil(V / 16)), 4 warps of 4 columns. RPL: rows of the state a lane holds, D <= 8 RPL. Lane i of the
-// eight that share a column holds rows 4 i + 32 j + (0 .. 3).
+// eight that share a column holds rows 4 i + 32 j + (0 .. 3). Four tokens a turn: with S the state the turn finds, G_j = g_0 ..
+// g_j and R_ji = g_(i+1) .. g_j (products, so that a vanishing decay is no division),
+//     u_j = beta_j (v_j - G_j S^T k_j - sum_(i<j) R_ji (k_i . k_j) u_i),   o_j = G_j S^T q_j + sum_(i<=j) R_ji (k_i . q_j) u_i,
+//     S <- G_3 S + sum_i R_3i k_i u_i,
+// which is the token-by-token recurrence written out: the eight sums over the state's rows are taken side by side. The factors
+// R_ji (k_i . k_j) and R_ji (k_i . q_j) do not depend on the column: each warp makes those of one turn of a staged chunk.
+#define DR_COEF 28          // floats a turn: 6 of keys on keys, 10 of keys on queries, G, R_3, beta
 template <int RPL>
 __global__ void __launch_bounds__(32 * DR_WARPS)
 delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state, const int* cu_q, const int* seq_pos0,
                   const int* seq_slot, int H, int G, int D, int V, int wide_qk, int wide_v) {
-    constexpr int DP = 8 * RPL, NJ = RPL / 4;
-    constexpr int STAGE = DR_NT * (2 * DP + DR_COLS + 4);          // k, q, v columns, (g, beta, k . q, -)
+    constexpr int DP = 8 * RPL, NJ = RPL / 4, TURNS = DR_NT / 4;
+    static_assert(TURNS == DR_WARPS, "a warp makes the factors of one turn of a chunk");
+    constexpr int STAGE = DR_NT * (2 * DP + DR_COLS + 2) + TURNS * DR_COEF;          // k, q, v columns, (g, beta), factors
     extern __shared__ __align__(16) float dr_smem[];
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DR_COLS, kh = h / (H / G);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, i8 = lane & 7;
@@ -151,21 +173,33 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
     auto fetch = [&](int c) {                     // chunk c into its stage
         float* base = dr_smem + (c % DR_STAGES) * STAGE;
         const int t0 = c * DR_NT, nt = min(DR_NT, n_tok - t0);
-        const float* src = qkv + (size_t)(r0 + t0) * C;
-        const int step = wide_qk ? 4 : 1, per = D / step;
-        for (int i = tid; i < 2 * nt * per; i += 32 * DR_WARPS) {
-            const int which = i / (nt * per), tt = i / per % nt, d = (i % per) * step;      // 0: k, 1: q
-            dr_cp(base + which * DR_NT * DP + tt * DP + d, src + (size_t)tt * C + (which ? 0 : G * D) + kh * D + d, wide_qk);
+        const float* src = qkv + (size_t)(r0 + t0) * C + kh * D;
+        constexpr int PER = DP / 4;
+#pragma unroll
+        for (int n = 0; n < 2 * DR_NT * PER / (32 * DR_WARPS); n++) {
+            const int i = tid + n * 32 * DR_WARPS;
+            const int which = i / (DR_NT * PER), tt = i / PER % DR_NT, d = (i % PER) * 4;      // 0: k, 1: q
+            if (tt >= nt || d >= D) continue;
+            float* to = base + (which * DR_NT + tt) * DP + d;
+            const float* from = src + (size_t)tt * C + (which ? 0 : G * D) + d;
+            if (wide_qk) dr_cp(to, from, true);
+            else
+                for (int e = 0; e < min(4, D - d); e++) dr_cp(to + e, from + e, false);
         }
-        const int vstep = wide_v ? 4 : 1, vper = n_cols / vstep;
-        for (int i = tid; i < nt * vper; i += 32 * DR_WARPS) {
-            const int tt = i / vper, d = (i % vper) * vstep;
-            dr_cp(base + 2 * DR_NT * DP + tt * DR_COLS + d, src + (size_t)tt * C + 2 * G * D + h * V + col0 + d, wide_v);
-        }
-        float* sc = base + DR_NT * (2 * DP + DR_COLS);
-        for (int i = tid; i < nt * 3; i += 32 * DR_WARPS) {
-            const int tt = i / 3, w = i % 3;
-            dr_cp(sc + tt * 4 + w, scal + (size_t)(r0 + t0 + tt) * nsc + (w == 0 ? h : w == 1 ? H + h : 2 * H + kh), false);
+        if (tid < DR_NT * DR_COLS / 4) {
+            const int tt = tid / (DR_COLS / 4), d = tid % (DR_COLS / 4) * 4;
+            if (tt < nt && d < n_cols) {
+                float* to = base + 2 * DR_NT * DP + tt * DR_COLS + d;
+                const float* from = qkv + (size_t)(r0 + t0 + tt) * C + 2 * G * D + h * V + col0 + d;
+                if (wide_v) dr_cp(to, from, true);
+                else
+                    for (int e = 0; e < min(4, n_cols - d); e++) dr_cp(to + e, from + e, false);
+            }
+        } else if (tid < DR_NT * DR_COLS / 4 + 2 * DR_NT) {
+            const int i = tid - DR_NT * DR_COLS / 4, tt = i / 2, w = i % 2;
+            float* to = base + DR_NT * (2 * DP + DR_COLS) + 2 * tt + w;
+            if (tt < nt) dr_cp(to, scal + (size_t)(r0 + t0 + tt) * nsc + (w == 0 ? h : H + h), false);
+            else *to = w == 0 ? 1.f : 0.f;         // tokens past the end: no decay and no step
         }
     };
     const int n_chunks = (n_tok + DR_NT - 1) / DR_NT;
@@ -189,45 +223,125 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
         __syncthreads();                           // chunk c is there, and every warp has left chunk c - 1
         if (c + DR_STAGES - 1 < n_chunks) fetch(c + DR_STAGES - 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        const float* base = dr_smem + (c % DR_STAGES) * STAGE;
+        float* base = dr_smem + (c % DR_STAGES) * STAGE;
+        float* coefs = base + DR_NT * (2 * DP + DR_COLS + 2);
+        {   // the factors of turn ``warp``
+            float d[16];
+#pragma unroll
+            for (int i = 0; i < 16; i++) d[i] = 0.f;
+#pragma unroll
+            for (int n = 0; n < (DP + 127) / 128; n++) {
+                const int at = 4 * lane + 128 * n;
+                if (at < DP) {
+                    float4 k[4];
+#pragma unroll
+                    for (int j = 0; j < 4; j++) k[j] = *reinterpret_cast<const float4*>(base + (4 * warp + j) * DP + at);
+                    auto dot = [](float acc, const float4& x, const float4& y) {
+                        return fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, acc))));
+                    };
+#pragma unroll
+                    for (int j = 0, n1 = 0, n2 = 6; j < 4; j++) {
+                        const float4 q = *reinterpret_cast<const float4*>(base + (DR_NT + 4 * warp + j) * DP + at);
+#pragma unroll
+                        for (int i = 0; i < j; i++, n1++) d[n1] = dot(d[n1], k[i], k[j]);
+#pragma unroll
+                        for (int i = 0; i <= j; i++, n2++) d[n2] = dot(d[n2], k[i], q);
+                    }
+                }
+            }
+            const float sum = dr_fold16(d, lane);
+            const float* gb = base + DR_NT * (2 * DP + DR_COLS) + 8 * warp;
+            const float g[4] = {gb[0], gb[2], gb[4], gb[6]};
+            const int idx = lane >> 1;
+            // (j, i) of the 16 values: keys on keys (1,0) (2,0) (2,1) (3,0) (3,1) (3,2), keys on queries (0,0) (1,0) (1,1) (2,0) .. (3,3)
+            const int j = (int)(0x3333222110333221ull >> (4 * idx)) & 15, i = (int)(0x3210210100210100ull >> (4 * idx)) & 15;
+            float r = 1.f;
+#pragma unroll
+            for (int m = 1; m < 4; m++)
+                if (m > i && m <= j) r *= g[m];
+            float* cf = coefs + warp * DR_COEF;
+            if ((lane & 1) == 0) cf[idx] = sum * r;
+            if (lane < 4) {
+                float up = 1.f, down = 1.f;
+#pragma unroll
+                for (int m = 0; m < 4; m++) {
+                    if (m <= lane) up *= g[m];
+                    if (m > lane) down *= g[m];
+                }
+                cf[16 + lane] = up, cf[20 + lane] = down, cf[24 + lane] = gb[2 * lane + 1];
+            }
+        }
+        __syncthreads();
         const float *ks = base + 4 * i8, *qs = ks + DR_NT * DP;
         const float* vs = base + 2 * DR_NT * DP + warp * 4 + (lane >> 3);
-        const float4* scs = reinterpret_cast<const float4*>(base + DR_NT * (2 * DP + DR_COLS));
         const int nt = min(DR_NT, n_tok - c * DR_NT);
-        float kn[RPL], qn[RPL];
-        auto rows_of = [&](int tt) {
-#pragma unroll
-            for (int j = 0; j < NJ; j++) {
-                const float4 x = *reinterpret_cast<const float4*>(ks + tt * DP + 32 * j);
-                const float4 y = *reinterpret_cast<const float4*>(qs + tt * DP + 32 * j);
-                kn[4 * j] = x.x, kn[4 * j + 1] = x.y, kn[4 * j + 2] = x.z, kn[4 * j + 3] = x.w;
-                qn[4 * j] = y.x, qn[4 * j + 1] = y.y, qn[4 * j + 2] = y.z, qn[4 * j + 3] = y.w;
-            }
-        };
-        rows_of(0);
-        for (int tt = 0; tt < nt; tt++) {
-            float kv[RPL], qv[RPL];
-#pragma unroll
-            for (int j = 0; j < RPL; j++) kv[j] = kn[j], qv[j] = qn[j];
-            const float4 g4 = scs[tt];
-            const float v = vs[tt * DR_COLS];
-            rows_of(min(tt + 1, nt - 1));
+#pragma unroll 1
+        for (int t0 = 0; t0 < nt; t0 += 4) {
             float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+            float kr[RPL <= 16 ? 4 : 1][RPL <= 16 ? RPL : 1];
 #pragma unroll
-            for (int j = 0; j < RPL; j++) {
-                a[j & 3] = fmaf(st[j], kv[j], a[j & 3]);
-                b[j & 3] = fmaf(st[j], qv[j], b[j & 3]);
+            for (int n = 0; n < NJ; n++) {
+                float4 k[4], q[4];
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    k[j] = *reinterpret_cast<const float4*>(ks + (t0 + j) * DP + 32 * n);
+                    q[j] = *reinterpret_cast<const float4*>(qs + (t0 + j) * DP + 32 * n);
+                }
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    a[j] = fmaf(st[4 * n], k[j].x, a[j]), b[j] = fmaf(st[4 * n], q[j].x, b[j]);
+                    a[j] = fmaf(st[4 * n + 1], k[j].y, a[j]), b[j] = fmaf(st[4 * n + 1], q[j].y, b[j]);
+                    a[j] = fmaf(st[4 * n + 2], k[j].z, a[j]), b[j] = fmaf(st[4 * n + 2], q[j].z, b[j]);
+                    a[j] = fmaf(st[4 * n + 3], k[j].w, a[j]), b[j] = fmaf(st[4 * n + 3], q[j].w, b[j]);
+                    if (RPL <= 16) {
+                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n) % (RPL <= 16 ? RPL : 1)] = k[j].x;
+                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n + 1) % (RPL <= 16 ? RPL : 1)] = k[j].y;
+                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n + 2) % (RPL <= 16 ? RPL : 1)] = k[j].z;
+                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n + 3) % (RPL <= 16 ? RPL : 1)] = k[j].w;
+                    }
+                }
             }
-            float as = (a[0] + a[1]) + (a[2] + a[3]), bs = (b[0] + b[1]) + (b[2] + b[3]);
+            float v[4];
 #pragma unroll
-            for (int off = 1; off < 8; off <<= 1) {
-                as += __shfl_xor_sync(0xffffffffu, as, off);
-                bs += __shfl_xor_sync(0xffffffffu, bs, off);
+            for (int j = 0; j < 4; j++) v[j] = vs[(t0 + j) * DR_COLS];
+            float cf[DR_COEF];
+#pragma unroll
+            for (int i = 0; i < DR_COEF; i += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(coefs + (t0 / 4) * DR_COEF + i);
+                cf[i] = x.x, cf[i + 1] = x.y, cf[i + 2] = x.z, cf[i + 3] = x.w;
             }
-            const float u = g4.y * (v - g4.x * as);
 #pragma unroll
-            for (int j = 0; j < RPL; j++) st[j] = fmaf(kv[j], u, g4.x * st[j]);
-            if (i8 == 0 && live) out[(size_t)(r0 + c * DR_NT + tt) * ow + (size_t)h * V + col] = fmaf(g4.z, u, g4.x * bs);
+            for (int off = 1; off < 8; off <<= 1)
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    a[j] += __shfl_xor_sync(0xffffffffu, a[j], off);
+                    b[j] += __shfl_xor_sync(0xffffffffu, b[j], off);
+                }
+            float u[4], o[4];
+#pragma unroll
+            for (int j = 0, n1 = 0, n2 = 6; j < 4; j++) {
+                float x = v[j] - cf[16 + j] * a[j];
+#pragma unroll
+                for (int i = 0; i < j; i++, n1++) x = fmaf(-cf[n1], u[i], x);
+                u[j] = cf[24 + j] * x;
+                o[j] = cf[16 + j] * b[j];
+#pragma unroll
+                for (int i = 0; i <= j; i++, n2++) o[j] = fmaf(cf[n2], u[i], o[j]);
+            }
+            const float w[4] = {cf[20] * u[0], cf[21] * u[1], cf[22] * u[2], cf[23] * u[3]};
+#pragma unroll
+            for (int n = 0; n < RPL; n++) {
+                float x = cf[19] * st[n];
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    const float k = RPL <= 16 ? kr[j % (RPL <= 16 ? 4 : 1)][n % (RPL <= 16 ? RPL : 1)] : ks[(t0 + j) * DP + 32 * (n / 4) + n % 4];
+                    x = fmaf(k, w[j], x);
+                }
+                st[n] = x;
+            }
+            // lane j of a column's eight stores token j
+            const float mine = i8 == 0 ? o[0] : i8 == 1 ? o[1] : i8 == 2 ? o[2] : o[3];
+            if (i8 < 4 && live && t0 + i8 < nt) out[(size_t)(r0 + c * DR_NT + t0 + i8) * ow + (size_t)h * V + col] = mine;
         }
     }
     if (live) {
@@ -364,7 +478,7 @@ DK_EXPORT int dk_delta_rule(const float* qkv, const float* scal, float* out, flo
     const dim3 grid(n_seq, H, (V + DR_COLS - 1) / DR_COLS), block(32 * DR_WARPS);
 #define DR_LAUNCH(R)                                                                                                           \
     if (D <= 8 * R) {                                                                                                          \
-        const size_t smem = sizeof(float) * DR_STAGES * DR_NT * (2 * 8 * R + DR_COLS + 4);                                     \
+        const size_t smem = sizeof(float) * DR_STAGES * (DR_NT * (2 * 8 * R + DR_COLS + 2) + DR_NT / 4 * DR_COEF);             \
         if (smem > 48 * 1024) cudaFuncSetAttribute(delta_rule_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         return dk_launch(delta_rule_kernel<R>, grid, block, smem, st, qkv, scal, out, state, cu_q, seq_pos0, seq_slot, H, G, D, V, \
                          wide_qk, wide_v);                                                                                     \

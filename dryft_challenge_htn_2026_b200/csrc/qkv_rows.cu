@@ -59,70 +59,124 @@ __device__ __forceinline__ void st_four(bf16* p, int d, int size, bool vec, cons
         if (d + e < size) p[d + e] = __float2bfloat16_rn(y[e]);
 }
 
-// y[i] holds coordinates 4 lane + 128 i .. + 3 of a head; the first ``dims`` coordinates turn by the table row (c, s)
-__device__ __forceinline__ void rotate_head(float (&y)[2][4], float* ys, const float* c, const float* s, int dims, int pairs) {
+// A lane's angles of a rotation over the first ``dims`` coordinates: its coordinates are 4 lane + 128 i + e. Pairs: the
+// angle of coordinate d is d / 2; halves: d below dims / 2, d - dims / 2 from there. Past the rotation: the identity.
+template <int NI>
+struct Angles {
+    float c[NI][4], s[NI][4];
+    __device__ __forceinline__ void load(const float* cosv, const float* sinv, int pos, int dims, int pairs) {
+        const int lane = threadIdx.x & 31, half = dims / 2;
+#pragma unroll
+        for (int i = 0; i < NI; i++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int d = 4 * lane + 128 * i + e, j = pairs ? d / 2 : d < half ? d : d - half;
+                const bool on = d < dims;
+                c[i][e] = on ? cosv[(size_t)pos * half + j] : 1.f;
+                s[i][e] = on ? sinv[(size_t)pos * half + j] : 0.f;
+            }
+    }
+};
+
+// y[i] holds coordinates 4 lane + 128 i .. + 3 of a head. Pairs turn inside a lane; halves meet their partner by a shuffle
+// where half the rotation is a multiple of four inside the first 128 coordinates, else through the warp's own shared memory.
+template <int NI>
+__device__ __forceinline__ void rotate_head(float (&y)[NI][4], float* ys, const Angles<NI>& a, int dims, int pairs) {
     const int lane = threadIdx.x & 31, half = dims / 2;
     if (pairs) {
 #pragma unroll
-        for (int i = 0; i < 2; i++)
+        for (int i = 0; i < NI; i++)
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
-                const int d = 4 * lane + 128 * i + e;
-                if (d < dims) {
-                    const float cc = c[d / 2], ss = s[d / 2], u = y[i][e], v = y[i][e + 1];
-                    y[i][e] = u * cc - v * ss;
-                    y[i][e + 1] = v * cc + u * ss;
-                }
+                const float u = y[i][e], v = y[i][e + 1];
+                y[i][e] = u * a.c[i][e] - v * a.s[i][e];
+                y[i][e + 1] = v * a.c[i][e] + u * a.s[i][e];
             }
+        return;
+    }
+    if (NI == 1 && half % 4 == 0) {
+        const bool low = 4 * lane < half;
+        const int from = low ? lane + half / 4 : lane - half / 4;
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const float other = __shfl_sync(0xffffffffu, y[0][e], from & 31);
+            y[0][e] = low ? y[0][e] * a.c[0][e] - other * a.s[0][e] : y[0][e] * a.c[0][e] + other * a.s[0][e];
+        }
         return;
     }
     __syncwarp();
 #pragma unroll
-    for (int i = 0; i < 2; i++)
+    for (int i = 0; i < NI; i++)
 #pragma unroll
         for (int e = 0; e < 4; e++) ys[4 * lane + 128 * i + e] = y[i][e];
     __syncwarp();
 #pragma unroll
-    for (int i = 0; i < 2; i++)
+    for (int i = 0; i < NI; i++)
 #pragma unroll
         for (int e = 0; e < 4; e++) {
             const int d = 4 * lane + 128 * i + e;
-            if (d < dims) {
-                const int j = d < half ? d : d - half;
-                const float cc = c[j], ss = s[j];
-                y[i][e] = d < half ? y[i][e] * cc - ys[d + half] * ss : y[i][e] * cc + ys[d - half] * ss;
-            }
+            if (d < dims) y[i][e] = d < half ? y[i][e] * a.c[i][e] - ys[d + half] * a.s[i][e] : y[i][e] * a.c[i][e] + ys[d - half] * a.s[i][e];
         }
 }
 
-template <typename T>
+// A block per token (and part of its heads); a warp takes up to HPW heads at a time, all of them asked for before any is
+// used. NI: 1 for heads up to 128, 2 up to 256.
+template <typename T, int NI, int HPW>
 __global__ void __launch_bounds__(32 * QR_WARPS)
 qkv_rows_kernel(const T* proj, long long ld, T* q_out, long long ldq, int norm_mode, const float* __restrict__ qn,
                 const float* __restrict__ kn, float eps, const float* __restrict__ cosv, const float* __restrict__ sinv,
                 int rot_dims, int pairs, const float* __restrict__ vcos, const float* __restrict__ vsin, int v_pairs,
                 const int* row_pos, const int* row_seq, int nh, int nkv, int hd, int hdv, T* k_store, T* v_store,
                 const int* page_table, int pt_stride, int vec) {
-    __shared__ float ys_all[QR_WARPS][256];
+    __shared__ float ys_all[QR_WARPS][128 * NI];
     __shared__ float2 sums[QR_WARPS];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
+    const int nq = nh * hd, nk = nkv * hd, heads = nh + 2 * nkv;
     pdl_wait();
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
+    const T* row = proj + (size_t)t * ld;
+    float y[HPW][NI][4];
+    auto load = [&](int head0) {
+#pragma unroll
+        for (int n = 0; n < HPW; n++) {
+            const int head = head0 + n * gridDim.y * QR_WARPS;
+            const bool is_v = head >= nh + nkv;
+            const T* src = row + (is_v ? nq + nk + (head - nh - nkv) * hdv : head * hd);
+#pragma unroll
+            for (int i = 0; i < NI; i++) ld_four<T>(src, 4 * lane + 128 * i, head >= heads ? 0 : is_v ? hdv : hd, vec, y[n][i]);
+        }
+    };
+    const int first = blockIdx.y * QR_WARPS + warp;
+    load(first);
     const int pos = row_pos[t];
     if (pos < 0) return;
-    const T* row = proj + (size_t)t * ld;
-    const int nq = nh * hd, nk = nkv * hd;
+    Angles<NI> ang, vang;
+    if (rot_dims > 0) ang.load(cosv, sinv, pos, rot_dims, pairs);
+    if (vcos != nullptr) vang.load(vcos, vsin, pos, hdv, v_pairs);
     float rq = 1.f, rk = 1.f;
     if (norm_mode == 3) {                          // all of q, and all of k, over their root mean squares
         float sq = 0.f, sk = 0.f;
-        for (int d = 4 * threadIdx.x; d < nq; d += 4 * 32 * QR_WARPS) {
-            float y[4];
-            ld_four<T>(row, d, nq, vec, y);
-            sq += (y[0] * y[0] + y[1] * y[1]) + (y[2] * y[2] + y[3] * y[3]);
-        }
-        for (int d = 4 * threadIdx.x; d < nk; d += 4 * 32 * QR_WARPS) {
-            float y[4];
-            ld_four<T>(row + nq, d, nk, vec, y);
-            sk += (y[0] * y[0] + y[1] * y[1]) + (y[2] * y[2] + y[3] * y[3]);
+        if (gridDim.y == 1 && heads <= HPW * QR_WARPS) {        // every head of the row is here already
+#pragma unroll
+            for (int n = 0; n < HPW; n++) {
+                const int head = first + n * QR_WARPS;
+                float ss = 0.f;
+#pragma unroll
+                for (int i = 0; i < NI; i++) ss += (y[n][i][0] * y[n][i][0] + y[n][i][1] * y[n][i][1]) + (y[n][i][2] * y[n][i][2] + y[n][i][3] * y[n][i][3]);
+                if (head < nh) sq += ss;
+                else if (head < nh + nkv) sk += ss;
+            }
+        } else {
+            for (int d = 4 * threadIdx.x; d < nq; d += 4 * 32 * QR_WARPS) {
+                float x[4];
+                ld_four<T>(row, d, nq, vec, x);
+                sq += (x[0] * x[0] + x[1] * x[1]) + (x[2] * x[2] + x[3] * x[3]);
+            }
+            for (int d = 4 * threadIdx.x; d < nk; d += 4 * 32 * QR_WARPS) {
+                float x[4];
+                ld_four<T>(row + nq, d, nk, vec, x);
+                sk += (x[0] * x[0] + x[1] * x[1]) + (x[2] * x[2] + x[3] * x[3]);
+            }
         }
         sq = warp_sum(sq), sk = warp_sum(sk);
         if (lane == 0) sums[warp] = make_float2(sq, sk);
@@ -135,54 +189,48 @@ qkv_rows_kernel(const T* proj, long long ld, T* q_out, long long ldq, int norm_m
     }
     const int page = k_store != nullptr ? page_table[(size_t)row_seq[t] * pt_stride + pos / DK_PAGE] : -1;
     float* ys = ys_all[warp];
-    const float *c = cosv + (size_t)pos * (rot_dims / 2), *s = sinv + (size_t)pos * (rot_dims / 2);
-    for (int head = blockIdx.y * QR_WARPS + warp; head < nh + 2 * nkv; head += gridDim.y * QR_WARPS) {
-        const bool is_q = head < nh, is_v = head >= nh + nkv;
-        if (!is_q && page < 0) continue;           // another layer's cache: only the queries are wanted
-        const int size = is_v ? hdv : hd;
-        const T* src = row + (is_v ? nq + nk + (head - nh - nkv) * hdv : head * hd);
-        float y[2][4];
+    for (int head0 = first;;) {
 #pragma unroll
-        for (int i = 0; i < 2; i++) ld_four<T>(src, 4 * lane + 128 * i, size, vec, y[i]);
-        if (is_v) {
-            if (vcos != nullptr) rotate_head(y, ys, vcos + (size_t)pos * (hdv / 2), vsin + (size_t)pos * (hdv / 2), hdv, v_pairs);
-        } else {
-            const float* w = is_q ? qn : kn;
-            if (norm_mode == 3) {
-                const float r = is_q ? rq : rk;
-                const int w0 = (is_q ? head : head - nh) * hd;
+        for (int n = 0; n < HPW; n++) {
+            const int head = head0 + n * gridDim.y * QR_WARPS;
+            if (head >= heads) break;
+            const bool is_q = head < nh, is_v = head >= nh + nkv;
+            if (!is_q && page < 0) continue;       // another layer's cache: only the queries are wanted
+            if (is_v) {
+                if (vcos != nullptr) rotate_head<NI>(y[n], ys, vang, hdv, v_pairs);
+            } else {
+                const float* w = is_q ? qn : kn;
+                auto scale = [&](float r, int w0) {
 #pragma unroll
-                for (int i = 0; i < 2; i++)
+                    for (int i = 0; i < NI; i++) {
+                        float ww[4] = {1.f, 1.f, 1.f, 1.f};
+                        if (w) ld_four<float>(w + w0, 4 * lane + 128 * i, hd, hd % 4 == 0, ww);
 #pragma unroll
-                    for (int e = 0; e < 4; e++) {
-                        const int d = 4 * lane + 128 * i + e;
-                        if (d < hd) y[i][e] *= w ? r * w[w0 + d] : r;
+                        for (int e = 0; e < 4; e++) y[n][i][e] *= r * ww[e];
                     }
+                };
+                auto norm_head = [&]() {
+                    float ss = 0.f;
+#pragma unroll
+                    for (int i = 0; i < NI; i++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) ss += y[n][i][e] * y[n][i][e];          // coordinates past the head are zero
+                    scale(1.f / sqrtf(warp_sum(ss) / (float)hd + eps), 0);
+                };
+                if (norm_mode == 3) scale(is_q ? rq : rk, (is_q ? head : head - nh) * hd);
+                if (norm_mode == 1) norm_head();
+                if (rot_dims > 0) rotate_head<NI>(y[n], ys, ang, rot_dims, pairs);
+                if (norm_mode == 2) norm_head();
             }
-            auto norm_head = [&]() {
-                float ss = 0.f;
+            T* dst = is_q ? q_out + (size_t)t * ldq + head * hd
+                          : is_v ? v_store + kv_offset(page, nkv, head - nh - nkv, pos % DK_PAGE, hdv)
+                                 : k_store + kv_offset(page, nkv, head - nh, pos % DK_PAGE, hd);
 #pragma unroll
-                for (int i = 0; i < 2; i++)
-#pragma unroll
-                    for (int e = 0; e < 4; e++) ss += y[i][e] * y[i][e];          // coordinates past the head are zero
-                const float r = 1.f / sqrtf(warp_sum(ss) / (float)hd + eps);
-#pragma unroll
-                for (int i = 0; i < 2; i++)
-#pragma unroll
-                    for (int e = 0; e < 4; e++) {
-                        const int d = 4 * lane + 128 * i + e;
-                        if (d < hd) y[i][e] *= w ? r * w[d] : r;
-                    }
-            };
-            if (norm_mode == 1) norm_head();
-            if (rot_dims > 0) rotate_head(y, ys, c, s, rot_dims, pairs);
-            if (norm_mode == 2) norm_head();
+            for (int i = 0; i < NI; i++) st_four(dst, 4 * lane + 128 * i, is_v ? hdv : hd, vec, y[n][i]);
         }
-        T* dst = is_q ? q_out + (size_t)t * ldq + head * hd
-                      : is_v ? v_store + kv_offset(page, nkv, head - nh - nkv, pos % DK_PAGE, hdv)
-                             : k_store + kv_offset(page, nkv, head - nh, pos % DK_PAGE, hd);
-#pragma unroll
-        for (int i = 0; i < 2; i++) st_four(dst, 4 * lane + 128 * i, size, vec, y[i]);
+        head0 += HPW * gridDim.y * QR_WARPS;
+        if (head0 >= heads) break;
+        load(head0);
     }
 }
 
@@ -250,16 +298,24 @@ DK_EXPORT int dk_qkv_rows(int dtype, const void* proj, long long ld, void* q_out
     // the heads of a row in one block where its norm spans them all, else dealt out so that few rows still fill the SMs
     const int groups = (nh + 2 * nkv + QR_WARPS - 1) / QR_WARPS;
     int split = 1;
-    if (norm_mode != 3) split = n_tok < 512 ? groups : (groups + 1) / 2;
+    if (norm_mode != 3) split = n_tok < 512 ? groups : (groups + 2) / 3;
     else if (n_tok <= 64) split = min(groups, 4);       // every block takes the sums anew: a short row read again
+    const int per = (groups + split - 1) / split;       // heads a warp
     const dim3 grid(n_tok, split), block(32 * QR_WARPS);
-    if (dtype == 0)
-        return dk_launch(qkv_rows_kernel<float>, grid, block, 0, st, (const float*)proj, ld, (float*)q_out, ldq, norm_mode, qn, kn,
-                         eps, cosv, sinv, rot_dims, pairs, vcos, vsin, v_pairs, row_pos, row_seq, nh, nkv, hd, hdv, (float*)k_store,
-                         (float*)v_store, page_table, pt_stride, vec);
-    return dk_launch(qkv_rows_kernel<bf16>, grid, block, 0, st, (const bf16*)proj, ld, (bf16*)q_out, ldq, norm_mode, qn, kn, eps,
-                     cosv, sinv, rot_dims, pairs, vcos, vsin, v_pairs, row_pos, row_seq, nh, nkv, hd, hdv, (bf16*)k_store,
-                     (bf16*)v_store, page_table, pt_stride, vec);
+#define QR_LAUNCH(T, NI, HPW)                                                                                                \
+    return dk_launch(qkv_rows_kernel<T, NI, HPW>, grid, block, 0, st, (const T*)proj, ld, (T*)q_out, ldq, norm_mode, qn, kn, eps, \
+                     cosv, sinv, rot_dims, pairs, vcos, vsin, v_pairs, row_pos, row_seq, nh, nkv, hd, hdv, (T*)k_store,      \
+                     (T*)v_store, page_table, pt_stride, vec)
+    const bool small = hd <= 128 && hdv <= 128;
+    if (dtype == 0) {
+        if (small) QR_LAUNCH(float, 1, 3);
+        QR_LAUNCH(float, 2, 2);
+    }
+    if (small && per <= 1) QR_LAUNCH(bf16, 1, 1);
+    if (small && per <= 3) QR_LAUNCH(bf16, 1, 3);
+    if (small) QR_LAUNCH(bf16, 1, 6);
+    QR_LAUNCH(bf16, 2, 2);
+#undef QR_LAUNCH
 }
 
 DK_EXPORT int dk_turn_back_gate(int dtype, const void* o, long long ldi, void* out, long long ldo, const void* gate, long long ldg,

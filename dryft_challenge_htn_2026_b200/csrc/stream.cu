@@ -147,34 +147,29 @@ __device__ __forceinline__ void load_source(float (&d)[NV][4], const Source<T>& 
         }
 }
 
-// v <- h[row] + norm(delta[row]); the stream as it stood goes to ``old_to`` when that is given
-template <typename T, int NV>
-__device__ __forceinline__ void summed_row(float (&v)[NV][4], const float* h, size_t row, const AddArgs<T>& a, int H, bool vec,
-                                           BlockSums& sums, float* old_to) {
+// v <- h[row] + norm(delta[row]): first the loads, which wait for nothing, ...
+template <typename T, int NV, bool TWO>
+__device__ __forceinline__ void load_row(float (&v)[NV][4], float (&d)[NV][4], float (&e)[TWO ? NV : 1][4], const float* h, size_t row,
+                                         const AddArgs<T>& a, int H, bool vec) {
 #pragma unroll
     for (int q = 0; q < NV; q++) ld_cols(h + row * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
-    if (old_to) {
-#pragma unroll
-        for (int q = 0; q < NV; q++) st_cols(old_to, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
-    }
+    if (a.s0.x || a.s0.parts) load_source<T, NV>(d, a.s0, row, H, vec);
+    if constexpr (TWO) load_source<T, NV>(e, a.s1, row, H, vec);
+}
+// ... then the norms and the sum
+template <typename T, int NV, bool TWO>
+__device__ __forceinline__ void sum_row(float (&v)[NV][4], float (&d)[NV][4], float (&e)[TWO ? NV : 1][4], const AddArgs<T>& a, int H, bool vec,
+                                        BlockSums& sums) {
     if (!a.s0.x && !a.s0.parts) return;
-    float d[NV][4];
-    load_source<T, NV>(d, a.s0, row, H, vec);
     if (a.s0.w) {
-        const bool two = a.s1.x || a.s1.parts;
-        float e[NV][4];
         float sd = 0.f, se = 0.f;
-        if (two) {
-            load_source<T, NV>(e, a.s1, row, H, vec);
-#pragma unroll
-            for (int q = 0; q < NV; q++)
-#pragma unroll
-                for (int k = 0; k < 4; k++) se += e[q][k] * e[q][k];
-        }
 #pragma unroll
         for (int q = 0; q < NV; q++)
 #pragma unroll
-            for (int k = 0; k < 4; k++) sd += d[q][k] * d[q][k];
+            for (int k = 0; k < 4; k++) {
+                sd += d[q][k] * d[q][k];
+                if constexpr (TWO) se += e[q][k] * e[q][k];
+            }
         const float2 t = sums(sd, se);
         const float rd = a.pre_scale / sqrtf(t.x / (float)H + a.pre_eps), re = a.pre_scale / sqrtf(t.y / (float)H + a.pre_eps);
 #pragma unroll
@@ -184,7 +179,7 @@ __device__ __forceinline__ void summed_row(float (&v)[NV][4], const float* h, si
             ld_cols(a.s0.w, c, H, vec, w);
 #pragma unroll
             for (int k = 0; k < 4; k++) d[q][k] *= rd * w[k];
-            if (two) {
+            if constexpr (TWO) {
                 ld_cols(a.s1.w, c, H, vec, w);
 #pragma unroll
                 for (int k = 0; k < 4; k++) d[q][k] = fmaf(e[q][k], re * w[k], d[q][k]);
@@ -198,8 +193,8 @@ __device__ __forceinline__ void summed_row(float (&v)[NV][4], const float* h, si
         for (int k = 0; k < 4; k++) v[q][k] += d[q][k];
 }
 
-template <typename T, int NV>
-__global__ void __launch_bounds__(NV > 4 ? 1024 : 512)
+template <typename T, int NV, bool TWO>
+__global__ void __launch_bounds__(NV == 1 || NV > 4 ? 1024 : 512)
 sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const int* rows, NormArgs next, T* a, float* save,
                     const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int H, int vec) {
     __shared__ float2 red[2][32];
@@ -207,13 +202,17 @@ sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const i
     pdl_wait();
     pdl_launch_dependents();
     const size_t out_row = blockIdx.x, row = rows ? (size_t)rows[out_row] : out_row;
-    float* old_to = nullptr;
+    float v[NV][4], d[NV][4], e[TWO ? NV : 1][4];
+    load_row<T, NV, TWO>(v, d, e, h, row, args, H, vec);
     if (save != nullptr && row_pos[row] >= 0) {
         const int s = row_seq[row];
-        if (cu_q == nullptr || (int)row + 1 == cu_q[s + 1]) old_to = save + (size_t)seq_slot[s] * H;
+        if (cu_q == nullptr || (int)row + 1 == cu_q[s + 1]) {
+            float* to = save + (size_t)seq_slot[s] * H;
+#pragma unroll
+            for (int q = 0; q < NV; q++) st_cols(to, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
+        }
     }
-    float v[NV][4];
-    summed_row<T, NV>(v, h, row, args, H, vec, sums, old_to);
+    sum_row<T, NV, TWO>(v, d, e, args, H, vec, sums);
     if (h_out != nullptr) {
 #pragma unroll
         for (int q = 0; q < NV; q++) st_cols(h_out + row * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
@@ -224,8 +223,8 @@ sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const i
     for (int q = 0; q < NV; q++) st_cols(a + out_row * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
 }
 
-template <typename T, int NV>
-__global__ void __launch_bounds__(NV > 4 ? 1024 : 512)
+template <typename T, int NV, bool TWO>
+__global__ void __launch_bounds__(NV == 1 || NV > 4 ? 1024 : 512)
 sublayer_add_shift_kernel(const float* h, float* h_out, const AddArgs<T> args, const float* __restrict__ share, const float* state,
                           const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int n_rows, int run,
                           T* a, int H, int vec) {
@@ -234,34 +233,39 @@ sublayer_add_shift_kernel(const float* h, float* h_out, const AddArgs<T> args, c
     pdl_wait();
     pdl_launch_dependents();
     const int r0 = blockIdx.x * run, r1 = min(n_rows, r0 + run);
-    float prev[NV][4];
+    float prev[NV][4], v[NV][4], d[NV][4], e[TWO ? NV : 1][4];
+    load_row<T, NV, TWO>(v, d, e, h, (size_t)r0, args, H, vec);
     for (int r = r0; r < r1; r++) {
         const int pos = row_pos[r];
         const int s = pos >= 0 ? row_seq[r] : 0;
+        const bool first = cu_q == nullptr || r == cu_q[s];
         if (pos < 0) {                                   // a padding row
 #pragma unroll
             for (int q = 0; q < NV; q++) prev[q][0] = prev[q][1] = prev[q][2] = prev[q][3] = 0.f;
-        } else if (cu_q == nullptr || r == cu_q[s]) {    // the first row its sequence brings: what the step before left
+        } else if (first) {                              // the first row its sequence brings: what the step before left
 #pragma unroll
             for (int q = 0; q < NV; q++)
                 ld_cols(state + (size_t)seq_slot[s] * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, prev[q]);
-        } else if (r == r0) {
-            summed_row<T, NV>(prev, h, (size_t)r - 1, args, H, vec, sums, nullptr);
+        } else if (r == r0) {                            // the row ahead of the block's run, worked out once more
+            float dp[NV][4], ep[TWO ? NV : 1][4];
+            load_row<T, NV, TWO>(prev, dp, ep, h, (size_t)r - 1, args, H, vec);
+            sum_row<T, NV, TWO>(prev, dp, ep, args, H, vec, sums);
         }
-        float v[NV][4];
-        summed_row<T, NV>(v, h, (size_t)r, args, H, vec, sums, nullptr);
+        sum_row<T, NV, TWO>(v, d, e, args, H, vec, sums);
+        float w[NV][4];
 #pragma unroll
         for (int q = 0; q < NV; q++) {
             const int c = (threadIdx.x + q * blockDim.x) * 4;
+            ld_cols(share, c, H, vec, w[q]);
             if (h_out != nullptr) st_cols(h_out + (size_t)r * H, c, H, vec, v[q]);
-            float w[4], o[4];
-            ld_cols(share, c, H, vec, w);
+            float o[4];
 #pragma unroll
-            for (int k = 0; k < 4; k++) o[k] = fmaf(prev[q][k] - v[q][k], w[k], v[q][k]);
+            for (int k = 0; k < 4; k++) o[k] = fmaf(prev[q][k] - v[q][k], w[q][k], v[q][k]);
             st_cols(a + (size_t)r * H, c, H, vec, o);
 #pragma unroll
             for (int k = 0; k < 4; k++) prev[q][k] = v[q][k];
         }
+        if (r + 1 < r1) load_row<T, NV, TWO>(v, d, e, h, (size_t)r + 1, args, H, vec);
     }
 }
 
@@ -306,9 +310,12 @@ __global__ void embed_bigram_kernel(const int* tok, const T* __restrict__ embed,
     for (int i = threadIdx.x; i < H; i += blockDim.x) h[(size_t)r * H + i] = fmaf(to_f(e[i]), scale, to_f(b[i]));
 }
 
-static inline int stream_threads(int H) {
+// Few rows (a decode step): every column of a row at once, four a thread. Many rows: fewer, longer threads, which leave room
+// for more blocks an SM.
+static inline int stream_threads(int H, int n_rows) {
     const int quads = (H + 3) / 4;
     if (quads > 2048) return 1024;
+    if (n_rows <= 256 && quads <= 1024) return (quads + 31) / 32 * 32;
     return quads > 1024 ? 512 : min(256, (quads + 31) / 32 * 32);
 }
 
@@ -341,17 +348,22 @@ DK_EXPORT int dk_sublayer_add(int dtype, const float* h, float* h_out, ADD_PARAM
                               float next_eps, int next_center, void* a, float* save, const int* row_pos, const int* row_seq,
                               const int* cu_q, const int* seq_slot, int n_rows, int H, cudaStream_t st) {
     if (H < 1 || H > 32768) return (int)cudaErrorInvalidValue;
-    const int threads = stream_threads(H), nv = ((H + 3) / 4 + threads - 1) / threads;
+    const int threads = stream_threads(H, n_rows), nv = ((H + 3) / 4 + threads - 1) / threads;
     const int vec = ADD_VEC && ((uintptr_t)next_w | (uintptr_t)save) % 16 == 0;
     const NormArgs next = {next_w, next_eps, next_center};
+    const bool two = x1 != nullptr || parts1 != nullptr;
+#define ADD_GO(NV, TWO)                                                                                                       \
+    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_kernel<T, NV, TWO>, dim3(n_rows), dim3(threads), 0, st, h, h_out,     \
+                                            make_add<T>(ADD_NAMES), rows, next, (T*)a, save, row_pos, row_seq, cu_q, seq_slot, \
+                                            H, vec))
 #define ADD_LAUNCH(NV)                                                                                                         \
-    if (nv <= NV && (threads <= 512 || NV == 8)) {                                                                                                            \
-        STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_kernel<T, NV>, dim3(n_rows), dim3(threads), 0, st, h, h_out,      \
-                                                make_add<T>(ADD_NAMES), rows, next, (T*)a, save, row_pos, row_seq, cu_q,       \
-                                                seq_slot, H, vec));                                                            \
+    if (nv <= NV && (threads <= 512 || NV == 1 || NV == 8)) {                                                                  \
+        if (two) ADD_GO(NV, true);                                                                                             \
+        ADD_GO(NV, false);                                                                                                     \
     }
     ADD_LAUNCH(1) ADD_LAUNCH(2) ADD_LAUNCH(3) ADD_LAUNCH(4) ADD_LAUNCH(8)
 #undef ADD_LAUNCH
+#undef ADD_GO
     return (int)cudaErrorInvalidValue;
 }
 
@@ -359,16 +371,21 @@ DK_EXPORT int dk_sublayer_add_shift(int dtype, const float* h, float* h_out, ADD
                                     const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int n_rows,
                                     int run, void* a, int H, cudaStream_t st) {
     if (H < 1 || H > 32768 || run < 1 || h == h_out) return (int)cudaErrorInvalidValue;
-    const int threads = stream_threads(H), nv = ((H + 3) / 4 + threads - 1) / threads;
+    const int threads = stream_threads(H, n_rows), nv = ((H + 3) / 4 + threads - 1) / threads;
     const int vec = ADD_VEC && ((uintptr_t)share | (uintptr_t)state) % 16 == 0;
+    const bool two = x1 != nullptr || parts1 != nullptr;
+#define ADD_GO(NV, TWO)                                                                                                       \
+    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_shift_kernel<T, NV, TWO>, dim3((n_rows + run - 1) / run),             \
+                                            dim3(threads), 0, st, h, h_out, make_add<T>(ADD_NAMES), share, state, row_pos,     \
+                                            row_seq, cu_q, seq_slot, n_rows, run, (T*)a, H, vec))
 #define ADD_LAUNCH(NV)                                                                                                         \
-    if (nv <= NV && (threads <= 512 || NV == 8)) {                                                                                                            \
-        STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_shift_kernel<T, NV>, dim3((n_rows + run - 1) / run), dim3(threads), \
-                                                0, st, h, h_out, make_add<T>(ADD_NAMES), share, state, row_pos, row_seq, cu_q, \
-                                                seq_slot, n_rows, run, (T*)a, H, vec));                                        \
+    if (nv <= NV && (threads <= 512 || NV == 1 || NV == 8)) {                                                                  \
+        if (two) ADD_GO(NV, true);                                                                                             \
+        ADD_GO(NV, false);                                                                                                     \
     }
     ADD_LAUNCH(1) ADD_LAUNCH(2) ADD_LAUNCH(3) ADD_LAUNCH(4) ADD_LAUNCH(8)
 #undef ADD_LAUNCH
+#undef ADD_GO
     return (int)cudaErrorInvalidValue;
 }
 
