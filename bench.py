@@ -1052,21 +1052,6 @@ def fukatar_kernel_times(torch, dk, pk, cfg_d, p_cfg):
                 gate, rot = proj[:, part.n_qkv:part.n_qkv + part.n_gate], part._rotation(ctx, part.value_position)
                 us = timed(lambda: api.turn_back_gate(mid, mid, gate, rot, 1.0, ctx.row_pos, s.num_heads, s.v_head_dim))
                 out[f"turn_back_gate_{tag}"] = bytes_rec(us, rows * part.n_mid * 2 * 2)
-        kv, H, D, L, Dv = cache.views(2)[0], ls.num_heads, ls.head_dim, ls.kv_rank, ls.v_head_dim
-        down = torch.randn(rows, lat.n_down + lat.n_fill, device=dev).to(bf)
-        table = ctx.tables[kv.group]
-        us = timed(lambda: api.latent_norm_rope_write(down[:, lat.n_q:lat.n_down], None, None, lat.kv_norm_w, ls.norm_eps, None, None, 0, ctx.row_pos,
-                                                      ctx.row_seq, 0, L, 0, kv.k, None, table))
-        out[f"latent_norm_cache_write_{tag}"] = bytes_rec(us, rows * L * 2 * 2)
-        ql = lat.queries(ctx, down[:, :lat.n_q])
-        us = timed(lambda: lat.queries(ctx, down[:, :lat.n_q]))
-        out[f"latent_query_heads_{tag}"] = flops_rec(us, 2 * rows * H * D * L) if pairs else bytes_rec(us, H * D * L * 2 + rows * (lat.n_q + H * L) * 2)
-        o_lat = torch.empty(rows, H * L, dtype=bf, device=dev)
-        us = timed(lambda: lat.core.attend(ctx, kv, ql, None, None, None, o_lat, 1.0, writes=False))
-        out[f"latent_attention_{tag}"] = flops_rec(us, 4 * H * L * pairs) if pairs else dict(bytes_rec(us, rows * keys * L * 2), keys=keys)
-        us = timed(lambda: lat.values(o_lat))
-        out[f"latent_value_heads_{tag}"] = flops_rec(us, 2 * rows * H * Dv * L) if pairs else bytes_rec(us, H * Dv * L * 2 + rows * (H * L + lat.n_mid) * 2)
-        del ql, o_lat, down
         # the recurrences: what a prompt must move (operands in float32 in, outputs out), what a single token must (the state, twice)
         proj = (torch.randn(rows, delta.n_in, device=dev) * 0.5).to(bf)
         mid = torch.empty(rows, delta.n_mid, dtype=bf, device=dev)
@@ -1091,6 +1076,21 @@ def fukatar_kernel_times(torch, dk, pk, cfg_d, p_cfg):
         us = timed(lambda: p_gla.mix(ctx, cache.views(3), pg, mg, 1.0))
         out[f"pibulix_gated_linear_attention_{tag}"] = bytes_rec(us, rows * gs.num_heads * (3 * gs.head_dim + 2 * gs.v_head_dim) * 4 if pairs else
                                                                  rows * gs.num_heads * gs.head_dim * gs.v_head_dim * 4 * 2)
+        kv, H, D, L, Dv = cache.views(2)[0], ls.num_heads, ls.head_dim, ls.kv_rank, ls.v_head_dim
+        down = torch.randn(rows, lat.n_down + lat.n_fill, device=dev).to(bf)
+        table = ctx.tables[kv.group]
+        us = timed(lambda: api.latent_norm_rope_write(down[:, lat.n_q:lat.n_down], None, None, lat.kv_norm_w, ls.norm_eps, None, None, 0, ctx.row_pos,
+                                                      ctx.row_seq, 0, L, 0, kv.k, None, table))
+        out[f"latent_norm_cache_write_{tag}"] = bytes_rec(us, rows * L * 2 * 2)
+        ql = lat.queries(ctx, down[:, :lat.n_q])
+        us = timed(lambda: lat.queries(ctx, down[:, :lat.n_q]))
+        out[f"latent_query_heads_{tag}"] = flops_rec(us, 2 * rows * H * D * L) if pairs else bytes_rec(us, H * D * L * 2 + rows * (lat.n_q + H * L) * 2)
+        o_lat = torch.empty(rows, H * L, dtype=bf, device=dev)
+        us = timed(lambda: lat.core.attend(ctx, kv, ql, None, None, None, o_lat, 1.0, writes=False))
+        out[f"latent_attention_{tag}"] = flops_rec(us, 4 * H * L * pairs) if pairs else dict(bytes_rec(us, rows * keys * L * 2), keys=keys)
+        us = timed(lambda: lat.values(o_lat))
+        out[f"latent_value_heads_{tag}"] = flops_rec(us, 2 * rows * H * Dv * L) if pairs else bytes_rec(us, H * Dv * L * 2 + rows * (H * L + lat.n_mid) * 2)
+        del ql, o_lat, down
         # the stream
         h, x, a = torch.randn(rows, W, device=dev), torch.empty(rows, W, device=dev), torch.randn(rows, W, device=dev).to(bf)
         b, o = torch.randn(rows, W, device=dev).to(bf), torch.empty(rows, W, dtype=bf, device=dev)

@@ -5,8 +5,8 @@
 //                      of q, k and v (its memory, the last taps - 1 projected rows, is a per-sequence state, read only
 //                      here), SiLU; q and k over sqrt(sum of squares + unit_eps) per head, q times D^(-1/2); g = exp(-exp(A)
 //                      softplus(a + dt)), beta = sigmoid(b); and k . q per key head (below).
-//   * delta_rule     : portions, four tokens a turn. Eight lanes share a column of the state, each with D / 8 of its rows in
-//                      registers for the whole portion; the rows q, k, v of 16 tokens at a time come through shared memory by
+//   * delta_rule     : portions, four tokens a turn. Eight lanes share a column of the state, its rows dealt
+//                      out over their registers for the whole portion; the rows q, k, v of 16 tokens at a time come through shared memory by
 //                      cp.async, three chunks in turn.
 //   * delta_rule_step: one token a sequence: a block per (sequence, head, 32 columns) passes once over its part of the state:
 //                      with a = S^T k and b = S^T q of the state as the token finds it, u = beta (v - g a), o = g b + (k . q) u.
@@ -16,8 +16,7 @@
 #define DP_THREADS 256
 #define DR_NT 16            // tokens a staged chunk
 #define DR_STAGES 3
-#define DR_WARPS 4
-#define DR_COLS (4 * DR_WARPS)
+#define DR_COLS 16          // columns of a state a block takes
 
 __device__ __forceinline__ float dr_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
@@ -121,6 +120,28 @@ delta_prepare_kernel(const T* proj, long long ld, const T* a_rows, const T* b_ro
     }
 }
 
+// two float32 multiply-adds an instruction (the halves of 64-bit registers), and their packing
+__device__ __forceinline__ uint64_t dr_fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t dr_mul2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ uint64_t dr_pack2(float lo, float hi) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 dr_unpack2(uint64_t x) {
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(x));
+    return d;
+}
+
 __device__ __forceinline__ void dr_cp(float* smem, const float* gmem, bool wide) {
     const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
     if (wide) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(gmem) : "memory");
@@ -142,26 +163,26 @@ __device__ __forceinline__ float dr_fold16(float (&d)[16], int lane) {
     return d[0] + __shfl_xor_sync(0xffffffffu, d[0], 1);
 }
 
-// grid (sequences, heads, ceil(V / 16)), 4 warps of 4 columns. RPL: rows of the state a lane holds, D <= 8 RPL. Lane i of the
-// eight that share a column holds rows 4 i + 32 j + (0 .. 3). Four tokens a turn: with S the state the turn finds, G_j = g_0 ..
+// grid (sequences, heads, ceil(V / 16)). LPC (8) lanes share a column of the state; lane i of them holds the RPL rows
+// 4 i + 4 LPC j + (0 .. 3), D <= LPC RPL. Four tokens a turn: with S the state the turn finds, G_j = g_0 ..
 // g_j and R_ji = g_(i+1) .. g_j (products, so that a vanishing decay is no division),
 //     u_j = beta_j (v_j - G_j S^T k_j - sum_(i<j) R_ji (k_i . k_j) u_i),   o_j = G_j S^T q_j + sum_(i<=j) R_ji (k_i . q_j) u_i,
 //     S <- G_3 S + sum_i R_3i k_i u_i,
 // which is the token-by-token recurrence written out: the eight sums over the state's rows are taken side by side. The factors
 // R_ji (k_i . k_j) and R_ji (k_i . q_j) do not depend on the column: each warp makes those of one turn of a staged chunk.
 #define DR_COEF 28          // floats a turn: 6 of keys on keys, 10 of keys on queries, G, R_3, beta
-template <int RPL>
-__global__ void __launch_bounds__(32 * DR_WARPS)
+template <int RPL, int LPC>
+__global__ void __launch_bounds__(LPC * DR_COLS)
 delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state, const int* cu_q, const int* seq_pos0,
                   const int* seq_slot, int H, int G, int D, int V, int wide_qk, int wide_v) {
-    constexpr int DP = 8 * RPL, NJ = RPL / 4, TURNS = DR_NT / 4;
-    static_assert(TURNS == DR_WARPS, "a warp makes the factors of one turn of a chunk");
+    constexpr int DP = LPC * RPL, NJ = RPL / 4, TURNS = DR_NT / 4, THREADS = LPC * DR_COLS;
+    static_assert(TURNS <= THREADS / 32, "a warp makes the factors of one turn of a chunk");
     constexpr int STAGE = DR_NT * (2 * DP + DR_COLS + 2) + TURNS * DR_COEF;          // k, q, v columns, (g, beta), factors
     extern __shared__ __align__(16) float dr_smem[];
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DR_COLS, kh = h / (H / G);
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, i8 = lane & 7;
-    const int col = col0 + warp * 4 + (lane >> 3);
-    for (int i = tid; i < DR_STAGES * STAGE; i += 32 * DR_WARPS) dr_smem[i] = 0.f;      // rows past D stay zero
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, il = lane % LPC;
+    const int col = col0 + tid / LPC;
+    for (int i = tid; i < DR_STAGES * STAGE; i += THREADS) dr_smem[i] = 0.f;      // rows past D stay zero
     pdl_wait();
     pdl_launch_dependents();
     if (seq_pos0[s] < 0) return;
@@ -176,10 +197,10 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
         const float* src = qkv + (size_t)(r0 + t0) * C + kh * D;
         constexpr int PER = DP / 4;
 #pragma unroll
-        for (int n = 0; n < 2 * DR_NT * PER / (32 * DR_WARPS); n++) {
-            const int i = tid + n * 32 * DR_WARPS;
+        for (int n = 0; n < (2 * DR_NT * PER + THREADS - 1) / THREADS; n++) {
+            const int i = tid + n * THREADS;
             const int which = i / (DR_NT * PER), tt = i / PER % DR_NT, d = (i % PER) * 4;      // 0: k, 1: q
-            if (tt >= nt || d >= D) continue;
+            if (which > 1 || tt >= nt || d >= D) continue;
             float* to = base + (which * DR_NT + tt) * DP + d;
             const float* from = src + (size_t)tt * C + (which ? 0 : G * D) + d;
             if (wide_qk) dr_cp(to, from, true);
@@ -210,14 +231,12 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
     }
     const bool live = col < V;
     float* S = state + (((size_t)seq_slot[s] * H + h) * D) * V + col;
-    float st[RPL];
+    uint64_t st[RPL / 2];                          // rows in pairs
 #pragma unroll
-    for (int j = 0; j < NJ; j++)
-#pragma unroll
-        for (int e = 0; e < 4; e++) {
-            const int d = 4 * i8 + 32 * j + e;
-            st[4 * j + e] = live && d < D ? S[(size_t)d * V] : 0.f;
-        }
+    for (int j = 0; j < RPL / 2; j++) {
+        const int d = 4 * il + 4 * LPC * (j / 2) + 2 * (j % 2);
+        st[j] = dr_pack2(live && d < D ? S[(size_t)d * V] : 0.f, live && d + 1 < D ? S[(size_t)(d + 1) * V] : 0.f);
+    }
     for (int c = 0; c < n_chunks; c++) {
         asm volatile("cp.async.wait_group %0;" ::"n"(DR_STAGES - 2) : "memory");
         __syncthreads();                           // chunk c is there, and every warp has left chunk c - 1
@@ -225,7 +244,7 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
         asm volatile("cp.async.commit_group;" ::: "memory");
         float* base = dr_smem + (c % DR_STAGES) * STAGE;
         float* coefs = base + DR_NT * (2 * DP + DR_COLS + 2);
-        {   // the factors of turn ``warp``
+        if (warp < TURNS) {   // the factors of turn ``warp``
             float d[16];
 #pragma unroll
             for (int i = 0; i < 16; i++) d[i] = 0.f;
@@ -272,34 +291,34 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
             }
         }
         __syncthreads();
-        const float *ks = base + 4 * i8, *qs = ks + DR_NT * DP;
-        const float* vs = base + 2 * DR_NT * DP + warp * 4 + (lane >> 3);
+        const float *ks = base + 4 * il, *qs = ks + DR_NT * DP;
+        const float* vs = base + 2 * DR_NT * DP + tid / LPC;
         const int nt = min(DR_NT, n_tok - c * DR_NT);
 #pragma unroll 1
         for (int t0 = 0; t0 < nt; t0 += 4) {
-            float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
-            float kr[RPL <= 16 ? 4 : 1][RPL <= 16 ? RPL : 1];
+            uint64_t a2[4] = {0, 0, 0, 0}, b2[4] = {0, 0, 0, 0};
+            constexpr bool KEEP = RPL <= 16;       // the keys stay in registers for the state's update
+            uint64_t kr[KEEP ? 4 : 1][KEEP ? RPL / 2 : 1];
 #pragma unroll
             for (int n = 0; n < NJ; n++) {
-                float4 k[4], q[4];
+                ulonglong2 k[4], q[4];
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
-                    k[j] = *reinterpret_cast<const float4*>(ks + (t0 + j) * DP + 32 * n);
-                    q[j] = *reinterpret_cast<const float4*>(qs + (t0 + j) * DP + 32 * n);
+                    k[j] = *reinterpret_cast<const ulonglong2*>(ks + (t0 + j) * DP + 4 * LPC * n);
+                    q[j] = *reinterpret_cast<const ulonglong2*>(qs + (t0 + j) * DP + 4 * LPC * n);
                 }
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
-                    a[j] = fmaf(st[4 * n], k[j].x, a[j]), b[j] = fmaf(st[4 * n], q[j].x, b[j]);
-                    a[j] = fmaf(st[4 * n + 1], k[j].y, a[j]), b[j] = fmaf(st[4 * n + 1], q[j].y, b[j]);
-                    a[j] = fmaf(st[4 * n + 2], k[j].z, a[j]), b[j] = fmaf(st[4 * n + 2], q[j].z, b[j]);
-                    a[j] = fmaf(st[4 * n + 3], k[j].w, a[j]), b[j] = fmaf(st[4 * n + 3], q[j].w, b[j]);
-                    if (RPL <= 16) {
-                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n) % (RPL <= 16 ? RPL : 1)] = k[j].x;
-                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n + 1) % (RPL <= 16 ? RPL : 1)] = k[j].y;
-                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n + 2) % (RPL <= 16 ? RPL : 1)] = k[j].z;
-                        kr[j % (RPL <= 16 ? 4 : 1)][(4 * n + 3) % (RPL <= 16 ? RPL : 1)] = k[j].w;
-                    }
+                    a2[j] = dr_fma2(st[2 * n], k[j].x, a2[j]), b2[j] = dr_fma2(st[2 * n], q[j].x, b2[j]);
+                    a2[j] = dr_fma2(st[2 * n + 1], k[j].y, a2[j]), b2[j] = dr_fma2(st[2 * n + 1], q[j].y, b2[j]);
+                    if constexpr (KEEP) kr[j][2 * n] = k[j].x, kr[j][2 * n + 1] = k[j].y;
                 }
+            }
+            float a[4], b[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float2 x = dr_unpack2(a2[j]), y = dr_unpack2(b2[j]);
+                a[j] = x.x + x.y, b[j] = y.x + y.y;
             }
             float v[4];
 #pragma unroll
@@ -311,7 +330,7 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
                 cf[i] = x.x, cf[i + 1] = x.y, cf[i + 2] = x.z, cf[i + 3] = x.w;
             }
 #pragma unroll
-            for (int off = 1; off < 8; off <<= 1)
+            for (int off = 1; off < LPC; off <<= 1)
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     a[j] += __shfl_xor_sync(0xffffffffu, a[j], off);
@@ -328,30 +347,35 @@ delta_rule_kernel(const float* qkv, const float* scal, float* out, float* state,
 #pragma unroll
                 for (int i = 0; i <= j; i++, n2++) o[j] = fmaf(cf[n2], u[i], o[j]);
             }
-            const float w[4] = {cf[20] * u[0], cf[21] * u[1], cf[22] * u[2], cf[23] * u[3]};
+            uint64_t w[4];
 #pragma unroll
-            for (int n = 0; n < RPL; n++) {
-                float x = cf[19] * st[n];
+            for (int j = 0; j < 4; j++) w[j] = dr_pack2(cf[20 + j] * u[j], cf[20 + j] * u[j]);
+            const uint64_t decay = dr_pack2(cf[19], cf[19]);
+#pragma unroll
+            for (int n = 0; n < RPL / 2; n++) {
+                uint64_t x = dr_mul2(decay, st[n]);
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
-                    const float k = RPL <= 16 ? kr[j % (RPL <= 16 ? 4 : 1)][n % (RPL <= 16 ? RPL : 1)] : ks[(t0 + j) * DP + 32 * (n / 4) + n % 4];
-                    x = fmaf(k, w[j], x);
+                    uint64_t k;
+                    if constexpr (KEEP) k = kr[j][n];
+                    else k = *reinterpret_cast<const uint64_t*>(ks + (t0 + j) * DP + 4 * LPC * (n / 2) + 2 * (n % 2));
+                    x = dr_fma2(k, w[j], x);
                 }
                 st[n] = x;
             }
-            // lane j of a column's eight stores token j
-            const float mine = i8 == 0 ? o[0] : i8 == 1 ? o[1] : i8 == 2 ? o[2] : o[3];
-            if (i8 < 4 && live && t0 + i8 < nt) out[(size_t)(r0 + c * DR_NT + t0 + i8) * ow + (size_t)h * V + col] = mine;
+            // lane j of a column stores token j
+            const float mine = il == 0 ? o[0] : il == 1 ? o[1] : il == 2 ? o[2] : o[3];
+            if (il < 4 && live && t0 + il < nt) out[(size_t)(r0 + c * DR_NT + t0 + il) * ow + (size_t)h * V + col] = mine;
         }
     }
     if (live) {
 #pragma unroll
-        for (int j = 0; j < NJ; j++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int d = 4 * i8 + 32 * j + e;
-                if (d < D) S[(size_t)d * V] = st[4 * j + e];
-            }
+        for (int j = 0; j < RPL / 2; j++) {
+            const int d = 4 * il + 4 * LPC * (j / 2) + 2 * (j % 2);
+            const float2 x = dr_unpack2(st[j]);
+            if (d < D) S[(size_t)d * V] = x.x;
+            if (d + 1 < D) S[(size_t)(d + 1) * V] = x.y;
+        }
     }
 }
 
@@ -475,15 +499,24 @@ DK_EXPORT int dk_delta_rule(const float* qkv, const float* scal, float* out, flo
     const int C = 2 * G * D + H * V;
     const int wide_qk = D % 4 == 0 && C % 4 == 0 && (uintptr_t)qkv % 16 == 0;
     const int wide_v = wide_qk && V % 4 == 0;
-    const dim3 grid(n_seq, H, (V + DR_COLS - 1) / DR_COLS), block(32 * DR_WARPS);
-#define DR_LAUNCH(R)                                                                                                           \
-    if (D <= 8 * R) {                                                                                                          \
-        const size_t smem = sizeof(float) * DR_STAGES * (DR_NT * (2 * 8 * R + DR_COLS + 2) + DR_NT / 4 * DR_COEF);             \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_rule_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        return dk_launch(delta_rule_kernel<R>, grid, block, smem, st, qkv, scal, out, state, cu_q, seq_pos0, seq_slot, H, G, D, V, \
-                         wide_qk, wide_v);                                                                                     \
+    const dim3 grid(n_seq, H, (V + DR_COLS - 1) / DR_COLS);
+    // Blocks that have an SM each must not share one: launched while the kernel before drains, they would pile up where it
+    // leaves first. More than half of an SM's shared memory keeps them apart.
+    int sms = 0, dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    const bool alone = (long long)grid.x * grid.y * grid.z <= sms;
+#define DR_LAUNCH(R, L)                                                                                                        \
+    if (D <= L * R) {                                                                                                          \
+        size_t smem = sizeof(float) * DR_STAGES * (DR_NT * (2 * L * R + DR_COLS + 2) + DR_NT / 4 * DR_COEF);             \
+        static bool attr = false;                                                                                              \
+        if (!attr) cudaFuncSetAttribute(delta_rule_kernel<R, L>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);     \
+        attr = true;                                                                                                           \
+        if (alone && smem < 116 * 1024) smem = 116 * 1024;                                                                     \
+        return dk_launch(delta_rule_kernel<R, L>, grid, dim3(L * DR_COLS), smem, st, qkv, scal, out, state, cu_q, seq_pos0,    \
+                         seq_slot, H, G, D, V, wide_qk, wide_v);                                                               \
     }
-    DR_LAUNCH(4) DR_LAUNCH(8) DR_LAUNCH(16) DR_LAUNCH(32)
+    DR_LAUNCH(4, 8) DR_LAUNCH(8, 8) DR_LAUNCH(16, 8) DR_LAUNCH(32, 8)
 #undef DR_LAUNCH
     return (int)cudaErrorInvalidValue;
 }

@@ -193,8 +193,8 @@ __device__ __forceinline__ void sum_row(float (&v)[NV][4], float (&d)[NV][4], fl
         for (int k = 0; k < 4; k++) v[q][k] += d[q][k];
 }
 
-template <typename T, int NV, bool TWO>
-__global__ void __launch_bounds__(NV == 1 || NV > 4 ? 1024 : 512)
+template <typename T, int NV, bool TWO, int MAXT>
+__global__ void __launch_bounds__(MAXT)
 sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const int* rows, NormArgs next, T* a, float* save,
                     const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int H, int vec) {
     __shared__ float2 red[2][32];
@@ -223,8 +223,8 @@ sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const i
     for (int q = 0; q < NV; q++) st_cols(a + out_row * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
 }
 
-template <typename T, int NV, bool TWO>
-__global__ void __launch_bounds__(NV == 1 || NV > 4 ? 1024 : 512)
+template <typename T, int NV, bool TWO, int MAXT>
+__global__ void __launch_bounds__(MAXT)
 sublayer_add_shift_kernel(const float* h, float* h_out, const AddArgs<T> args, const float* __restrict__ share, const float* state,
                           const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int n_rows, int run,
                           T* a, int H, int vec) {
@@ -234,38 +234,38 @@ sublayer_add_shift_kernel(const float* h, float* h_out, const AddArgs<T> args, c
     pdl_launch_dependents();
     const int r0 = blockIdx.x * run, r1 = min(n_rows, r0 + run);
     float prev[NV][4], v[NV][4], d[NV][4], e[TWO ? NV : 1][4];
-    load_row<T, NV, TWO>(v, d, e, h, (size_t)r0, args, H, vec);
-    for (int r = r0; r < r1; r++) {
-        const int pos = row_pos[r];
-        const int s = pos >= 0 ? row_seq[r] : 0;
-        const bool first = cu_q == nullptr || r == cu_q[s];
-        if (pos < 0) {                                   // a padding row
+    // whether row r is the first its sequence brings (or a padding row), so that its row before is not the one above
+    auto starts = [&](int r) { return row_pos[r] < 0 || cu_q == nullptr || r == cu_q[row_seq[r]]; };
+    bool first = starts(r0);
+    for (int r = first ? r0 : r0 - 1; r < r1; r++) {         // else the row ahead of the run is worked out once more
+        load_row<T, NV, TWO>(v, d, e, h, (size_t)r, args, H, vec);
+        const bool mine = r >= r0;
+        if (mine && r > r0) first = starts(r);
+        if (mine && first) {
+            if (row_pos[r] < 0) {
 #pragma unroll
-            for (int q = 0; q < NV; q++) prev[q][0] = prev[q][1] = prev[q][2] = prev[q][3] = 0.f;
-        } else if (first) {                              // the first row its sequence brings: what the step before left
+                for (int q = 0; q < NV; q++) prev[q][0] = prev[q][1] = prev[q][2] = prev[q][3] = 0.f;
+            } else {                                         // what the step before left
+                const float* st = state + (size_t)seq_slot[row_seq[r]] * H;
 #pragma unroll
-            for (int q = 0; q < NV; q++)
-                ld_cols(state + (size_t)seq_slot[s] * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, prev[q]);
-        } else if (r == r0) {                            // the row ahead of the block's run, worked out once more
-            float dp[NV][4], ep[TWO ? NV : 1][4];
-            load_row<T, NV, TWO>(prev, dp, ep, h, (size_t)r - 1, args, H, vec);
-            sum_row<T, NV, TWO>(prev, dp, ep, args, H, vec, sums);
+                for (int q = 0; q < NV; q++) ld_cols(st, (threadIdx.x + q * blockDim.x) * 4, H, vec, prev[q]);
+            }
         }
         sum_row<T, NV, TWO>(v, d, e, args, H, vec, sums);
-        float w[NV][4];
 #pragma unroll
         for (int q = 0; q < NV; q++) {
             const int c = (threadIdx.x + q * blockDim.x) * 4;
-            ld_cols(share, c, H, vec, w[q]);
-            if (h_out != nullptr) st_cols(h_out + (size_t)r * H, c, H, vec, v[q]);
-            float o[4];
+            if (mine) {
+                float w[4], o[4];
+                ld_cols(share, c, H, vec, w);
+                if (h_out != nullptr) st_cols(h_out + (size_t)r * H, c, H, vec, v[q]);
 #pragma unroll
-            for (int k = 0; k < 4; k++) o[k] = fmaf(prev[q][k] - v[q][k], w[q][k], v[q][k]);
-            st_cols(a + (size_t)r * H, c, H, vec, o);
+                for (int k = 0; k < 4; k++) o[k] = fmaf(prev[q][k] - v[q][k], w[k], v[q][k]);
+                st_cols(a + (size_t)r * H, c, H, vec, o);
+            }
 #pragma unroll
             for (int k = 0; k < 4; k++) prev[q][k] = v[q][k];
         }
-        if (r + 1 < r1) load_row<T, NV, TWO>(v, d, e, h, (size_t)r + 1, args, H, vec);
     }
 }
 
@@ -310,13 +310,13 @@ __global__ void embed_bigram_kernel(const int* tok, const T* __restrict__ embed,
     for (int i = threadIdx.x; i < H; i += blockDim.x) h[(size_t)r * H + i] = fmaf(to_f(e[i]), scale, to_f(b[i]));
 }
 
-// Few rows (a decode step): every column of a row at once, four a thread. Many rows: fewer, longer threads, which leave room
-// for more blocks an SM.
+// Few rows (a decode step): every column of a row at once, four a thread. Many rows: eight a thread, which leaves room for
+// more blocks an SM (up to 4,096 columns; wider rows take 512 threads).
 static inline int stream_threads(int H, int n_rows) {
     const int quads = (H + 3) / 4;
     if (quads > 2048) return 1024;
     if (n_rows <= 256 && quads <= 1024) return (quads + 31) / 32 * 32;
-    return quads > 1024 ? 512 : min(256, (quads + 31) / 32 * 32);
+    return quads > 1024 ? 512 : ((quads + 1) / 2 + 31) / 32 * 32;
 }
 
 #define STREAM_DISPATCH(dtype, ...)                     \
@@ -347,21 +347,21 @@ static AddArgs<T> make_add(const void* x0, const float* parts0, int n0, long lon
 DK_EXPORT int dk_sublayer_add(int dtype, const float* h, float* h_out, ADD_PARAMS, const int* rows, const float* next_w,
                               float next_eps, int next_center, void* a, float* save, const int* row_pos, const int* row_seq,
                               const int* cu_q, const int* seq_slot, int n_rows, int H, cudaStream_t st) {
-    if (H < 1 || H > 32768) return (int)cudaErrorInvalidValue;
+    if (H < 1 || H > 16384) return (int)cudaErrorInvalidValue;
     const int threads = stream_threads(H, n_rows), nv = ((H + 3) / 4 + threads - 1) / threads;
     const int vec = ADD_VEC && ((uintptr_t)next_w | (uintptr_t)save) % 16 == 0;
     const NormArgs next = {next_w, next_eps, next_center};
     const bool two = x1 != nullptr || parts1 != nullptr;
-#define ADD_GO(NV, TWO)                                                                                                       \
-    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_kernel<T, NV, TWO>, dim3(n_rows), dim3(threads), 0, st, h, h_out,     \
+#define ADD_GO(NV, TWO, MAXT)                                                                                                       \
+    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_kernel<T, NV, TWO, MAXT>, dim3(n_rows), dim3(threads), 0, st, h, h_out,     \
                                             make_add<T>(ADD_NAMES), rows, next, (T*)a, save, row_pos, row_seq, cu_q, seq_slot, \
                                             H, vec))
-#define ADD_LAUNCH(NV)                                                                                                         \
-    if (nv <= NV && (threads <= 512 || NV == 1 || NV == 8)) {                                                                  \
-        if (two) ADD_GO(NV, true);                                                                                             \
-        ADD_GO(NV, false);                                                                                                     \
+#define ADD_LAUNCH(NV, MAXT)                                                                                                         \
+    if (nv <= NV && threads <= MAXT) {                                                                  \
+        if (two) ADD_GO(NV, true, MAXT);                                                                                             \
+        ADD_GO(NV, false, MAXT);                                                                                                     \
     }
-    ADD_LAUNCH(1) ADD_LAUNCH(2) ADD_LAUNCH(3) ADD_LAUNCH(4) ADD_LAUNCH(8)
+    ADD_LAUNCH(1, 1024) ADD_LAUNCH(2, 512) ADD_LAUNCH(3, 512) ADD_LAUNCH(4, 512) ADD_LAUNCH(4, 1024)
 #undef ADD_LAUNCH
 #undef ADD_GO
     return (int)cudaErrorInvalidValue;
@@ -370,20 +370,20 @@ DK_EXPORT int dk_sublayer_add(int dtype, const float* h, float* h_out, ADD_PARAM
 DK_EXPORT int dk_sublayer_add_shift(int dtype, const float* h, float* h_out, ADD_PARAMS, const float* share, const float* state,
                                     const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int n_rows,
                                     int run, void* a, int H, cudaStream_t st) {
-    if (H < 1 || H > 32768 || run < 1 || h == h_out) return (int)cudaErrorInvalidValue;
+    if (H < 1 || H > 16384 || run < 1 || h == h_out) return (int)cudaErrorInvalidValue;
     const int threads = stream_threads(H, n_rows), nv = ((H + 3) / 4 + threads - 1) / threads;
     const int vec = ADD_VEC && ((uintptr_t)share | (uintptr_t)state) % 16 == 0;
     const bool two = x1 != nullptr || parts1 != nullptr;
-#define ADD_GO(NV, TWO)                                                                                                       \
-    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_shift_kernel<T, NV, TWO>, dim3((n_rows + run - 1) / run),             \
+#define ADD_GO(NV, TWO, MAXT)                                                                                                       \
+    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_shift_kernel<T, NV, TWO, MAXT>, dim3((n_rows + run - 1) / run),             \
                                             dim3(threads), 0, st, h, h_out, make_add<T>(ADD_NAMES), share, state, row_pos,     \
                                             row_seq, cu_q, seq_slot, n_rows, run, (T*)a, H, vec))
-#define ADD_LAUNCH(NV)                                                                                                         \
-    if (nv <= NV && (threads <= 512 || NV == 1 || NV == 8)) {                                                                  \
-        if (two) ADD_GO(NV, true);                                                                                             \
-        ADD_GO(NV, false);                                                                                                     \
+#define ADD_LAUNCH(NV, MAXT)                                                                                                         \
+    if (nv <= NV && threads <= MAXT) {                                                                  \
+        if (two) ADD_GO(NV, true, MAXT);                                                                                             \
+        ADD_GO(NV, false, MAXT);                                                                                                     \
     }
-    ADD_LAUNCH(1) ADD_LAUNCH(2) ADD_LAUNCH(3) ADD_LAUNCH(4) ADD_LAUNCH(8)
+    ADD_LAUNCH(1, 1024) ADD_LAUNCH(2, 512) ADD_LAUNCH(3, 512) ADD_LAUNCH(4, 512) ADD_LAUNCH(4, 1024)
 #undef ADD_LAUNCH
 #undef ADD_GO
     return (int)cudaErrorInvalidValue;
