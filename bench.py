@@ -964,14 +964,14 @@ def fukatar_config(width, heads, kv_heads, ff_qwen, layers, vocab):
     hd, h2, g2 = 128, heads // 2, max(1, kv_heads // 2)
     mlp = {"kind": "dense", "ff": 3 * ff_qwen // 2 // 64 * 64}
     par = {"type": "parallel",
-           "mixer": {"left": {"heads": h2, "kv_heads": g2, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 50.0, "rot": {"dims": hd // 2, "base": 1e4}},
+           "mixer": {"left": {"heads": h2, "kv_heads": g2, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 40.0, "rot": {"dims": hd // 2, "base": 5e5}},
                      "right": {"heads": h2, "kv_heads": h2 // 2, "dim": hd, "vdim": hd, "conv": 4}}, "mlp": mlp}
     att = {"type": "attention",
-           "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0,
+           "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 25.0,
                      "rot": {"dims": hd, "base": 1e6, "scaling": {"factor": 4.0, "original": 32768, "fast": 32.0, "slow": 1.0}}}, "mlp": mlp}
     lat = {"type": "latent_attention", "mixer": {"heads": heads, "dim": hd, "vdim": hd, "kv_rank": 512, "scale": hd ** -0.5}, "mlp": mlp}
     return dict(architecture="Fukatar", vocab=vocab, width=width, norm={"eps": 1e-6}, logit_softcap=30.0,
-                embedding={"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+                embedding={"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 127}},
                 layers=[(par, att, lat, lat)[i % 4] for i in range(layers)])
 
 

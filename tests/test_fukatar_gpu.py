@@ -206,7 +206,7 @@ def test_feed_forward_with_the_squared_relu(dtype, W, Fw):
 
 # ------------------------------------------------------------------------------------ positions
 @pytest.mark.parametrize("cls", [RotaryPartSpec, RotaryPairsSpec])
-@pytest.mark.parametrize("dims,base,scaling", [(16, 500.0, (4.0, 60, 8.0, 1.0)), (48, 50000.0, (2.0, 4096, 32.0, 1.0)), (2, 10.0, (3.0, 100, 1.0, 1.0)),
+@pytest.mark.parametrize("dims,base,scaling", [(16, 500.0, (4.0, 60, 8.0, 1.0)), (40, 30000.0, (2.5, 4096, 24.0, 1.0)), (2, 10.0, (3.0, 100, 1.0, 1.0)),
                                                (64, 1e6, (8.0, 100, 16.0, 2.0)), (22, 200.0, (1.0, 40, 1.0, 1.0)), (30, 7.0, None)])
 def test_angle_tables_of_stretched_positions(cls, dims, base, scaling):
     part = build_part(cls(dims, base, scaling), Runtime(DEV, torch.float32))
@@ -594,7 +594,7 @@ def random_config(rng):
     cfg = dict(architecture="Fukatar", vocab=rng.choice([50, 136, 333]), width=rng.choice([40, 52, 60, 100, 128, 160]),
                norm={"eps": rng.choice([1e-6, 1e-5, 1e-4])}, embedding={"scale": rng.choice([1.0, 4.0])}, layers=[one() for _ in range(rng.randint(2, 5))])
     if rng.random() < 0.8:
-        cfg["embedding"]["bigram"] = {"buckets": rng.choice([3, 64, 211]), "mul_prev": rng.choice([1, 31]), "mul_cur": rng.choice([1, 17])}
+        cfg["embedding"]["bigram"] = {"buckets": rng.choice([3, 64, 211]), "mul_prev": rng.choice([1, 29]), "mul_cur": rng.choice([1, 23])}
     if rng.random() < 0.7:
         cfg["logit_softcap"] = rng.choice([3.0, 30.0])
     return cfg
