@@ -53,11 +53,13 @@ class GroupRMSNormSpec:
 
 @dataclass(frozen=True)
 class LayerNormSpec:
-    """y = w * (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) over the last ``dim`` elements, no bias. ``tensor``: the
-    weight's name under the part's prefix (empty: the prefix itself names it)."""
+    """y = w * (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) over the last ``dim`` elements. ``tensor``: the
+    weight's name under the part's prefix (empty: the prefix itself names it). ``bias``: the name of a vector that is added
+    behind the weight (None: no bias)."""
     dim: int
     eps: float
     tensor: str = ""
+    bias: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -141,7 +143,8 @@ class MaskedAttentionSpec:
     the rotation. ``position`` may also be a ``RotaryPairsSpec``. ``value_position`` (a rotation spec over v_head_dim): the
     value of position j is turned by j and cached so, and each head's output at position i is turned back by i.
     ``head_gate``: each head's output times the one number sigmoid(W_g x)_h (tensor ``g`` [heads, hidden]), after the
-    turning back."""
+    turning back. ``keys_as_values``: there is no value projection (no tensor ``v``): a token's values are its keys as projected,
+    before their norm and rotation; the cache holds both."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -168,6 +171,7 @@ class MaskedAttentionSpec:
     qk_norm_whole: bool = False
     value_position: Optional[Any] = None
     head_gate: bool = False
+    keys_as_values: bool = False
 
 
 @dataclass(frozen=True)
@@ -295,6 +299,22 @@ class GatedLinearAttentionSpec:
 
 
 @dataclass(frozen=True)
+class MatrixMemorySpec:
+    """mLSTM: a matrix memory with exponential gates. q = W_q x * head_dim^(-1/2), k = W_k x (heads x head_dim), v = W_v x
+    (heads x v_head_dim); per head i = cap tanh((W_i x + b_i) / cap) and f = log sigmoid(cap tanh((W_f x + b_f) / cap)) with
+    cap = ``gate_cap``. Per head with the states S [head_dim, v_head_dim], n [head_dim] and m (all float32 and zero at the
+    start): m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T; n likewise with k alone; o = S^T q / (max(|n . q|,
+    e^(-m')) + 1e-6). Each head's o over its root mean square (``norm_eps`` inside the root), times ``norm`` (of all
+    heads' size), times sigmoid(W_g x), then ``o``."""
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    gate_cap: float
+    norm_eps: float
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Several mixers side by side on the same input; the result is the sum of scale_i * mixer_i(x).
     ``branches``: (checkpoint prefix under the mixer, mixer spec, scale) each. ``out_norm_eps``: each branch's output goes
@@ -336,7 +356,10 @@ class RoutedMLPSpec:
     themselves (times ``route_scale``); ``weight_on_input``: the weight multiplies the expert's input, out = sum
     expert(w x), not its output; ``shared_gate`` False: the shared expert is added as it is. ``activation`` "clamped":
     with g = min(gate x, limit), u = clamp(up x, -limit, limit) an expert is down(g sigmoid(1.702 g) (u + 1)), with
-    ``limit`` for the routed experts and ``shared_limit`` for the shared one."""
+    ``limit`` for the routed experts and ``shared_limit`` for the shared one. ``scores`` "softmax": s = softmax(W_router x)
+    over all router outputs. ``group_top``: how many of a group's largest choice scores (1 or 2) its own score sums.
+    ``identity``: that many router outputs more behind the experts': identity experts, which have no tensors and whose output
+    is the input itself; they take part in scores, groups and choice like the others."""
     hidden_size: int
     expert_ff: int
     num_experts: int
@@ -352,6 +375,9 @@ class RoutedMLPSpec:
     shared_gate: bool = True
     limit: Optional[float] = None
     shared_limit: Optional[float] = None
+    scores: str = "sigmoid"
+    group_top: int = 2
+    identity: int = 0
 
 
 @dataclass(frozen=True)
@@ -388,7 +414,8 @@ class PostNormLayerSpec:
 class SandwichLayerSpec:
     """One block with a norm before and after each sublayer: x <- x + norm_mix_out(mixer(norm_in(x))), then
     x <- x + norm_ff_out(feed_forward(norm_post(x))). Without a feed-forward the second step, its norms and their names
-    fall away."""
+    fall away. ``layer_scale``: names (under the prefix) of two vectors of the width that multiply what the two sublayers add,
+    behind their output norms, element by element."""
     prefix: str
     norm_in: Any
     mixer: Any
@@ -398,6 +425,7 @@ class SandwichLayerSpec:
     norm_ff_out: Any
     names: Tuple[Tuple[str, str], ...] = (("norm_in", "norm1."), ("mixer", "mix."), ("norm_mix_out", "norm1b."),
                                           ("norm_post", "norm2."), ("feed_forward", "mlp."), ("norm_ff_out", "norm2b."))
+    layer_scale: Optional[Tuple[str, str]] = None
 
 
 @dataclass(frozen=True)
@@ -433,12 +461,14 @@ class ScheduleEntry:
     """One run of a layer. ``cache`` names the cache entry the layer's mixer uses; with
     ``writes=False`` the mixer only reads what the entry's owner stored in this step. Right before the
     run the residual stream may take in the embedding's output once more (``add_embedding``) and a row
-    of a learned table of the model (``add_row`` = (name in ``ModelSpec.tables``, row))."""
+    of a learned table of the model (``add_row`` = (name in ``ModelSpec.tables``, row)). ``take_in`` (a name in
+    ``ModelSpec.matrices``): ahead of both, the stream x becomes M [x; x0] with x0 the embedding's output."""
     layer: int
     cache: int
     writes: bool = True
     add_embedding: bool = False
     add_row: Optional[Tuple[str, int]] = None
+    take_in: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -459,6 +489,7 @@ class ModelSpec:
     logit_cap: Optional[float] = None          # logits <- cap * tanh(logits / cap)
     logit_scale: float = 1.0                   # multiplies the logits before the cap
     tables: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()   # learned float32 tables of the model itself: (checkpoint name, shape)
+    matrices: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()  # learned matrices of the model itself: (checkpoint name, shape)
     embed_bigram: Optional[BigramSpec] = None  # rows of token pairs added to the (scaled) embedding
     unused_tensors: Tuple[str, ...] = ()       # checkpoint names the design ships although nothing reads them
     extra: dict = field(default_factory=dict, compare=False)

@@ -1237,14 +1237,15 @@ MOE_MAX_EXPERTS = 256
 
 
 def moe_route(x, w_router, correction, w_shared_gate, top, groups, keep, scale, idx, wt, shared_gate, scores=None,
-              renorm=True):
-    """Router of a mixture of experts, float32 arithmetic: s = sigmoid(w_router x); the ``top`` experts with the
-    largest s + correction among the ``keep`` best of ``groups`` groups of neighbours (group score: its two
-    largest s + correction) -> ``idx`` int32 [T, top]; ``wt`` float32 [T, top] = their s over the sum, times
+              renorm=True, softmax=False, group_top=2):
+    """Router of a mixture of experts, float32 arithmetic: s = sigmoid(w_router x), or with ``softmax`` the softmax of
+    w_router x; the ``top`` experts with the largest s + correction among the ``keep`` best of ``groups`` groups of
+    neighbours (group score: its ``group_top`` = 1 or 2 largest s + correction) -> ``idx`` int32 [T, top]; ``wt`` float32 [T, top] = their s over the sum, times
     ``scale`` (``renorm`` False: the chosen s themselves, times ``scale``; ``correction`` None: the choice goes by s);
     ``shared_gate`` float32 [T] = sigmoid(w_shared_gate . x) when that vector is given. Without a correction and with one
     group the choice goes by the sums w_router x themselves (the same order as their sigmoids, also where two float32
-    sigmoids have both reached 1), and ``scores`` then holds those sums. Two kernels: the
+    sigmoids have both reached 1), and ``scores`` then holds those sums (with ``softmax`` it always does, and with group
+    scores of one the choice goes by them whatever the groups). Two kernels: the
     scores (``scores`` float32 [T, E], scratch), then the choice."""
     _need(x, "x", None, 2), _need(w_router, "w_router", torch.float32, 2), _need(correction, "correction", torch.float32, 1)
     _need(w_shared_gate, "w_shared_gate", torch.float32, 1), _need(idx, "idx", torch.int32, 2), _need(wt, "wt", torch.float32, 2)
@@ -1253,7 +1254,8 @@ def moe_route(x, w_router, correction, w_shared_gate, top, groups, keep, scale, 
     E = w_router.shape[0]
     if w_router.shape[1] != W or idx.shape != (T, top) or wt.shape != (T, top) or E > MOE_MAX_EXPERTS or E % groups or \
             not 1 <= keep <= groups or not 1 <= top <= min(E, 32) or (correction is not None and correction.numel() != E) or \
-            (w_shared_gate is not None and (w_shared_gate.numel() != W or shared_gate is None or shared_gate.numel() != T)):
+            (w_shared_gate is not None and (w_shared_gate.numel() != W or shared_gate is None or shared_gate.numel() != T)) \
+            or group_top not in (1, 2):
         raise KernelError("moe_route: shapes do not match (up to 256 experts, up to 32 chosen)")
     if scores is None:
         scores = torch.empty((T, E), dtype=torch.float32, device=x.device)
@@ -1263,14 +1265,15 @@ def moe_route(x, w_router, correction, w_shared_gate, top, groups, keep, scale, 
     lib = _lib("moe.cu")
     _check(lib, lib.dk_moe_route(_dt(x), _p(x), W, _p(w_router), _p(correction), _p(w_shared_gate), E, int(top), int(groups),
                                  int(keep), c_float(scale), _p(idx), _p(wt), _p(shared_gate), _p(scores), T, int(bool(renorm)),
-                                 _stream()),
+                                 int(bool(softmax)), int(group_top), _stream()),
            "moe_route", 2)
 
 
 def moe_up_rows(x, w_gate_up, idx, mid, act=0, in_wt=None, limit=0.0):
     """mid[t * top + j] = act(gate_e x_t) * (up_e x_t) for e = idx[t, j]; w_gate_up [E, 2 ff, W] with an expert's
     gate rows before its up rows. A warp per output, float32 sums. ``in_wt`` float32 [T, top]: the pair's weight on the
-    expert's input (both sums times it before the activation). ``act`` ACT_CLAMPED with ``limit``: g' = min(g, limit),
+    expert's input (both sums times it before the activation). Numbers from E on are identity experts: their rows of
+    ``mid`` stay as they are. ``act`` ACT_CLAMPED with ``limit``: g' = min(g, limit),
     u' = clamp(u, -limit, limit), out = g' sigmoid(1.702 g') (u' + 1)."""
     _need(in_wt, "in_wt", torch.float32, 2)
     _need(x, "x", None, 2), _need(w_gate_up, "w_gate_up", x.dtype, 3), _need(idx, "idx", torch.int32, 2), _need(mid, "mid", x.dtype, 2)
@@ -1279,23 +1282,27 @@ def moe_up_rows(x, w_gate_up, idx, mid, act=0, in_wt=None, limit=0.0):
     if w_gate_up.shape[1:] != (2 * ff, W) or mid.shape[0] != T * top or idx.shape[0] != T:
         raise KernelError("moe_up_rows: shapes do not match")
     lib = _lib("moe.cu")
-    _check(lib, lib.dk_moe_up_rows(_dt(x), _p(x), W, _p(w_gate_up), _p(idx), _p(mid), ff, top, T, int(act), _p(in_wt),
+    _check(lib, lib.dk_moe_up_rows(_dt(x), _p(x), W, _p(w_gate_up), w_gate_up.shape[0], _p(idx), _p(mid), ff, top, T, int(act), _p(in_wt),
                                    c_float(limit), _stream()), "moe_up_rows")
 
 
-def moe_down_rows(mid, w_down, idx, wt, shared, shared_gate, out):
+def moe_down_rows(mid, w_down, idx, wt, shared, shared_gate, out, x=None, in_wt=None):
     """out[t] = sum_j wt[t, j] * down_e mid[t * top + j] (e = idx[t, j]) + shared_gate[t] * shared[t]; w_down
-    [E, W, ff]; ``shared`` [T, W] and its gate optional."""
+    [E, W, ff]; ``shared`` [T, W] and its gate optional. An e from E on is an identity expert: its output is ``x``[t]
+    (``in_wt``: the pair's weight, where it stands on the expert's input). ``x`` is needed where there are such experts."""
+    _need(x, "x", mid.dtype, 2), _need(in_wt, "in_wt", torch.float32, 2)
     _need(mid, "mid", None, 2), _need(w_down, "w_down", mid.dtype, 3), _need(idx, "idx", torch.int32, 2)
     _need(wt, "wt", torch.float32, 2), _need(shared, "shared", mid.dtype, 2), _need(shared_gate, "shared_gate", torch.float32, 1)
     _need(out, "out", mid.dtype, 2)
     T, top = idx.shape
     W, ff = w_down.shape[1:]
+    if x is not None and x.shape != (T, W):
+        raise KernelError("moe_down_rows: shapes do not match")
     if mid.shape != (T * top, ff) or out.shape != (T, W) or (wt is not None and wt.shape != (T, top)) or (shared is not None and shared.shape != (T, W)):
         raise KernelError("moe_down_rows: shapes do not match")
     lib = _lib("moe.cu")
-    _check(lib, lib.dk_moe_down_rows(_dt(mid), _p(mid), _p(w_down), _p(idx), _p(wt), _p(shared), _p(shared_gate), _p(out), W, ff,
-                                     top, T, _stream()), "moe_down_rows")
+    _check(lib, lib.dk_moe_down_rows(_dt(mid), _p(mid), _p(w_down), w_down.shape[0], _p(idx), _p(wt), _p(shared), _p(shared_gate),
+                                     _p(x), _p(in_wt), _p(out), W, ff, top, T, _stream()), "moe_down_rows")
 
 
 MOE_TILE_ROWS = 64
@@ -1311,7 +1318,8 @@ def moe_experts_tiles(x, w_gate_up, w_down, idx, wt, shared, shared_gate, out, a
     """The routed experts for many tokens: pairs sorted by expert on the device, tiles of 64 pairs as matrix
     products on mma.sync tensor cores (gate/up with the activation, then down), then the weighted sum per token
     plus shared_gate * shared. ``scratch(key, make)``: where buffers that outlive the call may be kept. ``wt`` None: the
-    plain sum; ``in_wt``, ``limit``: as in ``moe_up_rows``."""
+    plain sum; ``in_wt``, ``limit``: as in ``moe_up_rows``. Numbers in ``idx`` from E on are identity experts: their output
+    is the token's row of ``x``."""
     _need(in_wt, "in_wt", torch.float32, 2)
     _need(x, "x", torch.bfloat16, 2), _need(w_gate_up, "w_gate_up", torch.bfloat16, 3), _need(w_down, "w_down", torch.bfloat16, 3)
     _need(idx, "idx", torch.int32, 2), _need(wt, "wt", torch.float32, 2), _need(shared, "shared", torch.bfloat16, 2)
@@ -1337,7 +1345,7 @@ def moe_experts_tiles(x, w_gate_up, w_down, idx, wt, shared, shared_gate, out, a
     _check(lib, lib.dk_moe_up_tiles(_p(x), _p(w_gate_up), _p(tiles), max_tiles, _p(perm), top, _p(mid), ff, W, int(act), _p(in_wt),
                                     c_float(limit), _stream()), "moe_up_tiles")
     _check(lib, lib.dk_moe_down_tiles(_p(mid), _p(w_down), _p(tiles), max_tiles, _p(y), W, ff, _stream()), "moe_down_tiles")
-    _check(lib, lib.dk_moe_sum(_p(y), _p(inv), _p(wt), _p(shared), _p(shared_gate), _p(out), T, W, top, _stream()), "moe_sum")
+    _check(lib, lib.dk_moe_sum(_p(y), _p(inv), _p(wt), _p(shared), _p(shared_gate), _p(x), _p(in_wt), _p(out), T, W, top, _stream()), "moe_sum")
 
 
 def gated_linear_attention_takes_warps(head_dim, v_head_dim):
@@ -1606,8 +1614,9 @@ class NormedSum:
 
 
 def _add_args(h, delta, norm, dtype, what):
-    """The C arguments of what joins the stream: sources, their norms, the norm of their sum. ``norm``: None or (weight, eps,
-    center)."""
+    """The C arguments of what joins the stream ``h`` (or what has its shape): sources, their norms, the norm of their sum.
+    ``norm``: as ``_norm_args`` takes it."""
+    width = h.shape[1]
     normed = isinstance(delta, NormedSum)
     sources = delta.deltas if normed else [] if delta is None else [delta]
     args = []
@@ -1620,12 +1629,17 @@ def _add_args(h, delta, norm, dtype, what):
         if (src is not None and tuple(src.shape) != tuple(h.shape)) or (w is not None and w.numel() != h.shape[1]):
             raise KernelError(f"{what}: shapes do not match")
         args += [_p(x), parts, n, stride if src is not None else c_longlong(0), _p(w)]
-    nw, eps, center = norm if norm is not None else (None, 0.0, False)
-    _need(nw, "norm weight", torch.float32, 1)
-    if nw is not None and nw.numel() != h.shape[1]:
-        raise KernelError(f"{what}: shapes do not match")
-    return args + [c_float(delta.eps if normed else 0.0), c_float(delta.factor if normed else 1.0), _p(nw), c_float(eps),
-                   int(bool(center))]
+    return args + [c_float(delta.eps if normed else 0.0), c_float(delta.factor if normed else 1.0)] + _norm_args(norm, width, what)
+
+
+def _norm_args(norm, width, what):
+    """The C arguments of a norm given as None, (weight, eps, center) or (weight, eps, center, bias or None)."""
+    w, eps, center, b = (None, 0.0, False, None) if norm is None else tuple(norm) + ((None,) if len(norm) == 3 else ())
+    for t in (w, b):
+        _need(t, "norm weight", torch.float32, 1)
+        if t is not None and t.numel() != width:
+            raise KernelError(f"{what}: shapes do not match")
+    return [_p(w), _p(b), c_float(eps), int(bool(center))]
 
 
 def _need_sequences(row_pos, row_seq, cu_q, seq_slot, rows):
@@ -1635,26 +1649,34 @@ def _need_sequences(row_pos, row_seq, cu_q, seq_slot, rows):
         raise KernelError("positions and sequences of every row are needed")
 
 
-def sublayer_add(h, delta, norm, a_out, h_out=None, rows=None, next_norm=None, save=None, seqs=None):
-    """h_out = h + norm(delta) (float32), a_out = that row in its own type, or ``next_norm`` of it. ``delta``: None, a tensor,
-    a ``Partial`` or a ``NormedSum``; ``norm`` and ``next_norm``: None or (weight, eps, center), center True for a layer norm.
+def sublayer_add(h, delta, norm, a_out, h_out=None, rows=None, next_norm=None, save=None, seqs=None, base=None):
+    """h_out = h + norm(delta) (float32), a_out (rows of a wider matrix, maybe; None: not wanted) = that row in its own type, or
+    ``next_norm`` of it. ``delta``: None, a tensor, a ``Partial`` or a ``NormedSum``; ``norm`` and ``next_norm``: None or
+    (weight, eps, center) or (weight, eps, center, bias), center True for a layer norm. ``h`` None: the stream starts anew,
+    h_out = base + norm(delta) with ``base`` a float32 vector [H] or None (zero).
     ``rows`` (int32): a_out row i is made of h row rows[i], h_out is not written. ``save`` (float32 [slots, H]): h as it stood
     before the sum goes there at every sequence's last row, ``seqs`` = (row_pos, row_seq, cu_q or None, seq_slot)."""
-    _need(h, "h", torch.float32, 2), _need(h_out, "h_out", torch.float32, 2), _need(a_out, "a_out", None, 2)
-    _need(rows, "rows", torch.int32, 1), _need(save, "save", torch.float32, 2)
+    _need(h, "h", torch.float32, 2), _need(h_out, "h_out", torch.float32, 2), _need_rows(a_out, "a_out")
+    _need(rows, "rows", torch.int32, 1), _need(save, "save", torch.float32, 2), _need(base, "base", torch.float32, 1)
+    stream = h
+    if h is None:
+        h = h_out if h_out is not None else delta
+        if h is None or rows is not None or save is not None:
+            raise KernelError("sublayer_add: a stream that starts anew has no rows to gather and nothing to save")
     n = h.shape[0] if rows is None else rows.numel()
-    if tuple(a_out.shape) != (n, h.shape[1]) or (h_out is not None and (h_out.shape != h.shape or rows is not None)) \
+    if (a_out is not None and tuple(a_out.shape) != (n, h.shape[1])) or (a_out is None and h_out is None) or \
+            (base is not None and (stream is not None or base.numel() != h.shape[1])) or (h_out is not None and (h_out.shape != h.shape or rows is not None)) \
             or (save is not None and (seqs is None or save.shape[1] != h.shape[1] or rows is not None)):
         raise KernelError("sublayer_add: shapes do not match")
-    args = _add_args(h, delta, norm, a_out.dtype, "sublayer_add")
-    nw, neps, ncenter = next_norm if next_norm is not None else (None, 0.0, False)
-    _need(nw, "next norm weight", torch.float32, 1)
+    dtype = a_out.dtype if a_out is not None else delta.dtype if isinstance(delta, torch.Tensor) else torch.float32
+    args = _add_args(h, delta, norm, dtype, "sublayer_add")
     row_pos, row_seq, cu_q, seq_slot = seqs if seqs is not None else (None,) * 4
     if save is not None:
         _need_sequences(row_pos, row_seq, cu_q, seq_slot, h.shape[0])
     lib = _lib("stream.cu")
-    _check(lib, lib.dk_sublayer_add(_dt(a_out), _p(h), _p(h_out), *args, _p(rows), _p(nw), c_float(neps), int(bool(ncenter)),
-                                    _p(a_out), _p(save), _p(row_pos), _p(row_seq), _p(cu_q), _p(seq_slot), n, h.shape[1],
+    _check(lib, lib.dk_sublayer_add(0 if dtype == torch.float32 else 1, _p(stream), _p(base), _p(h_out), *args, _p(rows),
+                                    *_norm_args(next_norm, h.shape[1], "sublayer_add"), _p(a_out),
+                                    c_longlong(a_out.stride(0) if a_out is not None else 0), _p(save), _p(row_pos), _p(row_seq), _p(cu_q), _p(seq_slot), n, h.shape[1],
                                     _stream()), "sublayer_add")
 
 
@@ -1709,8 +1731,8 @@ NORM_WHOLE = 3
 
 
 def qkv_rows(proj, q_out, norm_mode, q_norm_w, k_norm_w, eps, rot, v_rot, row_pos, row_seq, n_heads, n_kv_heads, head_dim, v_head_dim,
-             k_store=None, v_store=None, page_table=None):
-    """Rows [q | k | v] of a projection -> ``q_out`` [tokens, heads * head_dim] and, with the paged stores, each token's k and
+             k_store=None, v_store=None, page_table=None, keys_as_values=False):
+    """Rows [q | k | v] of a projection, or [q | k] with ``keys_as_values`` (a token's values are its k columns as they are) -> ``q_out`` [tokens, heads * head_dim] and, with the paged stores, each token's k and
     v heads at their place there. ``norm_mode``: NORM_NONE, NORM_BEFORE_ROTATION, NORM_AFTER_ROTATION (per head, weights of
     the head's size or None) or NORM_WHOLE (all heads at once before the rotation, weights of the whole projection's size or
     None). ``rot`` and ``v_rot``: None or (cos, sin [positions, dims / 2], dims, pairs): the rotation of the first ``dims``
@@ -1725,7 +1747,8 @@ def qkv_rows(proj, q_out, norm_mode, q_norm_w, k_norm_w, eps, rot, v_rot, row_po
             if r[2] % 2 or r[2] > limit or r[0].shape[1] != r[2] // 2 or r[1].shape != r[0].shape:
                 raise KernelError(f"qkv_rows: {nm} over {r[2]} coordinates of {limit}")
     sizes = (n_q, n_k) if norm_mode == NORM_WHOLE else (head_dim, head_dim)
-    if proj.shape[1] != n_q + n_k + n_kv_heads * v_head_dim or q_out.shape != (proj.shape[0], n_q) or max(head_dim, v_head_dim) > 256 \
+    if proj.shape[1] != n_q + n_k + (0 if keys_as_values else n_kv_heads * v_head_dim) or (keys_as_values and head_dim != v_head_dim) \
+            or q_out.shape != (proj.shape[0], n_q) or max(head_dim, v_head_dim) > 256 \
             or any(w is not None and w.numel() != n for w, n in zip((q_norm_w, k_norm_w), sizes)) \
             or (v_rot is not None and v_rot[2] != v_head_dim):
         raise KernelError("qkv_rows: shapes do not match")
@@ -1740,7 +1763,7 @@ def qkv_rows(proj, q_out, norm_mode, q_norm_w, k_norm_w, eps, rot, v_rot, row_po
                                 _p(q_norm_w), _p(k_norm_w), c_float(eps), _p(cos), _p(sin), int(dims), int(bool(pairs)), _p(vcos),
                                 _p(vsin), int(bool(v_pairs)), _p(row_pos), _p(row_seq), proj.shape[0], n_heads, n_kv_heads, head_dim,
                                 v_head_dim, _p(k_store), _p(v_store), _p(page_table),
-                                page_table.shape[1] if page_table is not None else 0, _stream()), "qkv_rows")
+                                page_table.shape[1] if page_table is not None else 0, int(bool(keys_as_values)), _stream()), "qkv_rows")
 
 
 def turn_back_gate(o, out, gate, v_rot, out_scale, row_pos, n_heads, v_head_dim):
@@ -1809,3 +1832,52 @@ def delta_rule(qkv, scal, out, state, cu_q, seq_pos0, seq_slot, n_seq, n_heads, 
     else:
         _check(lib, lib.dk_delta_rule(_p(qkv), _p(scal), _p(out), _p(state), _p(cu_q), _p(seq_pos0), _p(seq_slot), n_seq, n_heads,
                                       n_kv_heads, head_dim, v_head_dim, _stream()), "delta_rule")
+
+
+# ---------------------------------------------------------------------------------- matrix memory with exponential gates
+def _need_memory(q, k, v, i_rows, f_rows, i_bias, f_bias, states, n_heads, head_dim, v_head_dim, what):
+    for t, nm in ((q, "q"), (k, "k"), (v, "v"), (i_rows, "i_rows"), (f_rows, "f_rows")):
+        _need_rows(t, nm, q.dtype)
+    _need(i_bias, "i_bias", torch.float32, 1), _need(f_bias, "f_bias", torch.float32, 1)
+    for t, nm, shape in zip(states, ("state", "n_state", "m_state"), ((n_heads, head_dim, v_head_dim), (n_heads, head_dim), (n_heads,))):
+        _need(t, nm, torch.float32)
+        if tuple(t.shape[1:]) != shape:
+            raise KernelError(f"{what}: {nm} must be [slots, {shape}]")
+    T = q.shape[0]
+    if not (q.stride(0) == k.stride(0) == v.stride(0) == i_rows.stride(0) == f_rows.stride(0)) or k.shape != q.shape \
+            or q.shape[1] != n_heads * head_dim or v.shape != (T, n_heads * v_head_dim) or i_rows.shape != (T, n_heads) \
+            or f_rows.shape != (T, n_heads) or i_bias.numel() != n_heads or f_bias.numel() != n_heads or not 1 <= head_dim <= 256:
+        raise KernelError(f"{what}: shapes do not match (columns of one matrix, key sizes up to 256)")
+
+
+def matrix_memory(q, k, v, gate, i_rows, f_rows, i_bias, f_bias, cap, states, weight, eps, out_scale, out, q_scale, cu_q, seq_pos0, seq_slot,
+                  row_pos, n_seq, n_heads, head_dim, v_head_dim):
+    """The matrix memory with exponential gates over a step's rows, all float32 behind the projection: log gates i = cap
+    tanh((i_rows + i_bias) / cap), f = log sigmoid of the same form; m' = max(f + m, i); S <- exp(f + m - m') S + exp(i - m')
+    k v^T, n likewise with k alone; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6) with q times ``q_scale``; ``out`` = each head's
+    o over its root mean square (``eps`` inside the root) * ``weight`` [heads * v_head_dim] * sigmoid(gate) * ``out_scale``.
+    ``states`` = (S [slots, heads, D, V], n [slots, heads, D], m [slots, heads]), float32, moved on. Rows of sequence s are
+    cu_q[s] .. cu_q[s + 1]; ``cu_q`` None: row s alone, seq_pos0[s] < 0 marks padding. Single tokens are one kernel, portions
+    three (gates, recurrence, output)."""
+    _need_memory(q, k, v, i_rows, f_rows, i_bias, f_bias, states, n_heads, head_dim, v_head_dim, "matrix_memory")
+    _need_rows(gate, "gate", q.dtype), _need_rows(out, "out", q.dtype), _need(weight, "weight", torch.float32, 1)
+    for t, nm in ((cu_q, "cu_q"), (seq_pos0, "seq_pos0"), (seq_slot, "seq_slot"), (row_pos, "row_pos")):
+        _need(t, nm, torch.int32, 1)
+    T, n_mid = q.shape[0], n_heads * v_head_dim
+    if gate.shape != (T, n_mid) or out.shape != (T, n_mid) or weight.numel() != n_mid or gate.stride(0) != q.stride(0) or not cap > 0:
+        raise KernelError("matrix_memory: shapes do not match, or a cap that is not positive")
+    S, n, m = states
+    lib, ld = _lib("matrix_memory.cu"), c_longlong(q.stride(0))
+    sizes = (n_heads, head_dim, v_head_dim)
+    if cu_q is None:
+        return _check(lib, lib.dk_mm_step(_dt(q), _p(q), _p(k), _p(v), _p(gate), _p(i_rows), _p(f_rows), ld, _p(i_bias), _p(f_bias), c_float(cap),
+                                          _p(S), _p(n), _p(m), _p(weight), c_float(eps), c_float(out_scale), _p(out), c_longlong(out.stride(0)),
+                                          _p(seq_pos0), _p(seq_slot), c_float(q_scale), T, *sizes, _stream()), "matrix_memory")
+    scal = torch.empty((T, n_heads, 4), dtype=torch.float32, device=q.device)
+    o = torch.empty((T, n_mid), dtype=torch.float32, device=q.device)
+    _check(lib, lib.dk_mm_gates(_dt(q), _p(i_rows), _p(f_rows), ld, _p(i_bias), _p(f_bias), c_float(cap), _p(scal), _p(m), _p(cu_q), _p(seq_pos0),
+                                _p(seq_slot), n_seq, n_heads, _stream()), "matrix_memory gates")
+    _check(lib, lib.dk_mm_portion(_dt(q), _p(q), _p(k), _p(v), ld, _p(scal), _p(o), _p(S), _p(n), _p(cu_q), _p(seq_pos0), _p(seq_slot),
+                                  c_float(q_scale), n_seq, *sizes, _stream()), "matrix_memory")
+    _check(lib, lib.dk_mm_output(_dt(q), _p(o), _p(scal), _p(weight), c_float(eps), _p(gate), ld, c_float(out_scale), _p(out),
+                                 c_longlong(out.stride(0)), _p(row_pos), T, n_heads, v_head_dim, _stream()), "matrix_memory output")

@@ -1,10 +1,11 @@
 // Mixture of experts: the router and the routed experts' feed-forward.
 //
-// Router (float32 throughout): z = W_r x, s = sigmoid(z); the choice is made on s + correction, among the
-// experts of the `keep` best of `groups` equal groups of neighbouring experts (a group's score is the sum of
-// its two largest choice scores; the others' choice scores count as minus infinity), the `top` largest;
-// the weights are the chosen experts' s (without the correction) over their sum, times a constant. The same
-// kernel works out the gate of a shared expert, sigmoid(w_sg . x), one number a token.
+// Router (float32 throughout): z = W_r x, s = sigmoid(z) or softmax(z); the choice is made on s + correction, among the
+// experts of the `keep` best of `groups` equal groups of neighbouring experts (a group's score is its largest choice
+// score, or the sum of its two largest; the others' choice scores count as minus infinity), the `top` largest;
+// the weights are the chosen experts' s (without the correction), also over their sum, times a constant. The same
+// kernel works out the gate of a shared expert, sigmoid(w_sg . x), one number a token. Router outputs behind the last
+// expert are identity experts: they have no matrices, their output is the token's row itself.
 //
 // Experts, row form (this file): every (token, chosen expert) pair is a row of its own,
 //   mid[pair] = act(W_gate[e] x) * (W_up[e] x),   out[token] = sum_j weight_j W_down[e_j] mid[pair_j]
@@ -97,7 +98,7 @@ moe_scores_kernel(const T* x, int W, const float* __restrict__ wr, const float* 
 // Choice: a warp a token, from the token's scores.
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
 moe_choose_kernel(const float* scores, const float* __restrict__ corr, int E, int top, int groups, int keep, float scale,
-                  int* idx, float* wt, int n_tok, int renorm, int by_logit) {
+                  int* idx, float* wt, int n_tok, int renorm, int by_logit, int softmax, int group_top) {
     extern __shared__ __align__(16) unsigned char route_smem[];
     pdl_wait();
     pdl_launch_dependents();
@@ -109,7 +110,9 @@ moe_choose_kernel(const float* scores, const float* __restrict__ corr, int E, in
     float* gs = c + E;
     for (int e = lane; e < E; e += 32) {
         const float v = scores[(size_t)t * E + e];
-        if (by_logit) {      // no correction, one group: the largest scores are the largest sums, and two float32 scores that
+        if (softmax) {
+            s[e] = v;
+        } else if (by_logit) {      // no correction, one group: the largest scores are the largest sums, and two float32 scores that
                              // have both reached 1 still differ in their sums
             s[e] = 1.f / (1.f + expf(-v));
             c[e] = v;
@@ -119,15 +122,32 @@ moe_choose_kernel(const float* scores, const float* __restrict__ corr, int E, in
         }
     }
     __syncwarp();
+    if (softmax) {           // over all of the token's sums
+        float top_z = -INFINITY, sum = 0.f;
+        for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, s[e]);
+        top_z = warp_max(top_z);
+        for (int e = lane; e < E; e += 32) {
+            const float z = s[e], p = expf(z - top_z);
+            s[e] = p;
+            c[e] = z;        // without a correction the choice goes by the sums (scores may have vanished where these still differ)
+            sum += p;
+        }
+        const float inv = 1.f / warp_sum(sum);
+        for (int e = lane; e < E; e += 32) {
+            s[e] *= inv;
+            if (!by_logit) c[e] = s[e] + (corr ? corr[e] : 0.f);
+        }
+        __syncwarp();
+    }
     if (groups > 1 && keep < groups) {
         const int per = E / groups;
-        for (int g = lane; g < groups; g += 32) {       // a group's score: its two largest choice scores
+        for (int g = lane; g < groups; g += 32) {       // a group's score: its largest choice score, or the two largest
             float a = -INFINITY, b = -INFINITY;
             for (int i = 0; i < per; i++) {
                 const float v = c[g * per + i];
                 if (v > a) { b = a; a = v; } else if (v > b) b = v;
             }
-            gs[g] = per > 1 ? a + b : a;
+            gs[g] = per > 1 && group_top > 1 ? a + b : a;
         }
         __syncwarp();
         // the keep best groups are marked by +inf; all others' experts then leave the choice
@@ -203,13 +223,14 @@ template <> struct Vec<float> {
 // boundaries), several requests in flight, or element by element for other widths.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(128)
-moe_up_rows_kernel(const T* x, int W, const T* __restrict__ wgu, const int* idx, T* mid, int ff, int top, int rows_per_block,
+moe_up_rows_kernel(const T* x, int W, const T* __restrict__ wgu, int E, const int* idx, T* mid, int ff, int top, int rows_per_block,
                    int act, const float* in_wt, float limit) {
     extern __shared__ float xs[];
     pdl_wait();
     pdl_launch_dependents();
     const int pair = blockIdx.x, t = pair / top;
     const int e = idx[pair];
+    if (e >= E) return;                              // an identity expert
     for (int k = threadIdx.x; k < W; k += blockDim.x) xs[k] = to_f(x[(size_t)t * W + k]);
     __syncthreads();
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
@@ -250,17 +271,19 @@ moe_up_rows_kernel(const T* x, int W, const T* __restrict__ wgu, const int* idx,
     }
 }
 
-// Block (token, slice of the width): out[t][c] = sum_j wt[t][j] (W_d[e_j][c] . mid[t*top + j]) + sgate[t] * shared[t][c].
+// Block (token, slice of the width): out[t][c] = sum_j wt[t][j] (W_d[e_j][c] . mid[t*top + j]) + sgate[t] * shared[t][c];
+// an identity expert (e_j at least E) gives wt[t][j] x[t][c] (in_wt: the weight stood on the input).
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(128)
-moe_down_rows_kernel(const T* mid, const T* __restrict__ wd, const int* idx, const float* wt, const T* shared,
-                     const float* sgate, T* out, int W, int ff, int top, int rows_per_block) {
+moe_down_rows_kernel(const T* mid, const T* __restrict__ wd, int E, const int* idx, const float* wt, const T* shared,
+                     const float* sgate, const T* x, const float* in_wt, T* out, int W, int ff, int top, int rows_per_block) {
     extern __shared__ float ms[];        // [top][ff], already times the pair's weight
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
     for (int i = threadIdx.x; i < top * ff; i += blockDim.x)
-        ms[i] = to_f(mid[(size_t)t * top * ff + i]) * (wt != nullptr ? wt[(size_t)t * top + i / ff] : 1.f);
+        if (idx[(size_t)t * top + i / ff] < E)
+            ms[i] = to_f(mid[(size_t)t * top * ff + i]) * (wt != nullptr ? wt[(size_t)t * top + i / ff] : 1.f);
     __syncthreads();
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
     const int c_end = min(W, (int)(blockIdx.y + 1) * rows_per_block);
@@ -268,6 +291,11 @@ moe_down_rows_kernel(const T* mid, const T* __restrict__ wd, const int* idx, con
     for (int c = blockIdx.y * rows_per_block + w; c < c_end; c += 4) {
         float acc = 0.f;
         for (int j = 0; j < top; j++) {
+            if (idx[(size_t)t * top + j] >= E) {
+                const float* w = wt != nullptr ? wt : in_wt;
+                if (lane == 0) acc = fmaf(w != nullptr ? w[(size_t)t * top + j] : 1.f, to_f(x[(size_t)t * W + c]), acc);
+                continue;
+            }
             const T* row = wd + ((size_t)idx[(size_t)t * top + j] * W + c) * ff;
             float a = 0.f;
             if (VEC) {
@@ -307,60 +335,61 @@ static int launch_scores(const void* x, int W, const float* wr, const float* wsg
 // scores: float32 scratch [n_tok, E]
 DK_EXPORT int dk_moe_route(int dtype, const void* x, int W, const float* wr, const float* corr, const float* wsg, int E,
                            int top, int groups, int keep, float scale, int* idx, float* wt, float* sgate, float* scores, int n_tok,
-                           int renorm, cudaStream_t st) {
+                           int renorm, int softmax, int group_top, cudaStream_t st) {
     if (E < 1 || E > MOE_MAX_EXPERTS || top < 1 || top > 32 || top > E || groups < 1 || E % groups || keep < 1 || keep > groups ||
         scores == nullptr || (sizeof(float) * ROUTE_TOKENS * W > 200 * 1024))
         return (int)cudaErrorInvalidValue;
-    const int by_logit = corr == nullptr && groups == 1;
-    int e = dtype == 0 ? launch_scores<float>(x, W, wr, wsg, E, scores, sgate, n_tok, by_logit, st)
-                       : launch_scores<bf16>(x, W, wr, wsg, E, scores, sgate, n_tok, by_logit, st);
+    const int by_logit = corr == nullptr && (groups == 1 || (softmax && group_top == 1));
+    const int sums = by_logit || softmax;        // what the first kernel leaves: the sums themselves, or their sigmoids
+    int e = dtype == 0 ? launch_scores<float>(x, W, wr, wsg, E, scores, sgate, n_tok, sums, st)
+                       : launch_scores<bf16>(x, W, wr, wsg, E, scores, sgate, n_tok, sums, st);
     if (e) return e;
     const size_t smem = sizeof(float) * 3 * (size_t)E * ROUTE_WARPS;
     return dk_launch(moe_choose_kernel, dim3((n_tok + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(32 * ROUTE_WARPS), smem, st, scores, corr,
-                     E, top, groups, keep, scale, idx, wt, n_tok, renorm, by_logit);
+                     E, top, groups, keep, scale, idx, wt, n_tok, renorm, by_logit, softmax, group_top);
 }
 
 template <typename T, bool VEC>
-static int launch_up(const void* x, int W, const void* wgu, const int* idx, void* mid, int ff, int top, int n_tok, int act,
+static int launch_up(const void* x, int W, const void* wgu, int E, const int* idx, void* mid, int ff, int top, int n_tok, int act,
                      const float* in_wt, float limit, cudaStream_t st) {
     const int rpb = 16;
     const dim3 grid(n_tok * top, (ff + rpb - 1) / rpb), block(128);
     const size_t smem = sizeof(float) * (size_t)W;
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_up_rows_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return dk_launch(moe_up_rows_kernel<T, VEC>, grid, block, smem, st, (const T*)x, W, (const T*)wgu, idx, (T*)mid, ff, top, rpb, act,
+    return dk_launch(moe_up_rows_kernel<T, VEC>, grid, block, smem, st, (const T*)x, W, (const T*)wgu, E, idx, (T*)mid, ff, top, rpb, act,
                      in_wt, limit);
 }
 
 template <typename T, bool VEC>
-static int launch_down(const void* mid, const void* wd, const int* idx, const float* wt, const void* shared, const float* sgate,
-                       void* out, int W, int ff, int top, int n_tok, cudaStream_t st) {
+static int launch_down(const void* mid, const void* wd, int E, const int* idx, const float* wt, const void* shared, const float* sgate,
+                       const void* x, const float* in_wt, void* out, int W, int ff, int top, int n_tok, cudaStream_t st) {
     const int rpb = 16;
     const dim3 grid(n_tok, (W + rpb - 1) / rpb), block(128);
     const size_t smem = sizeof(float) * (size_t)top * ff;
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_down_rows_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return dk_launch(moe_down_rows_kernel<T, VEC>, grid, block, smem, st, (const T*)mid, (const T*)wd, idx, wt, (const T*)shared,
-                     sgate, (T*)out, W, ff, top, rpb);
+    return dk_launch(moe_down_rows_kernel<T, VEC>, grid, block, smem, st, (const T*)mid, (const T*)wd, E, idx, wt, (const T*)shared,
+                     sgate, (const T*)x, in_wt, (T*)out, W, ff, top, rpb);
 }
 
-DK_EXPORT int dk_moe_up_rows(int dtype, const void* x, int W, const void* wgu, const int* idx, void* mid, int ff, int top,
+DK_EXPORT int dk_moe_up_rows(int dtype, const void* x, int W, const void* wgu, int E, const int* idx, void* mid, int ff, int top,
                              int n_tok, int act, const float* in_wt, float limit, cudaStream_t st) {
     const bool vec = (uintptr_t)wgu % 16 == 0 && W % (dtype == 0 ? 4 : 8) == 0;
     if (dtype == 0)
-        return vec ? launch_up<float, true>(x, W, wgu, idx, mid, ff, top, n_tok, act, in_wt, limit, st)
-                   : launch_up<float, false>(x, W, wgu, idx, mid, ff, top, n_tok, act, in_wt, limit, st);
-    return vec ? launch_up<bf16, true>(x, W, wgu, idx, mid, ff, top, n_tok, act, in_wt, limit, st)
-               : launch_up<bf16, false>(x, W, wgu, idx, mid, ff, top, n_tok, act, in_wt, limit, st);
+        return vec ? launch_up<float, true>(x, W, wgu, E, idx, mid, ff, top, n_tok, act, in_wt, limit, st)
+                   : launch_up<float, false>(x, W, wgu, E, idx, mid, ff, top, n_tok, act, in_wt, limit, st);
+    return vec ? launch_up<bf16, true>(x, W, wgu, E, idx, mid, ff, top, n_tok, act, in_wt, limit, st)
+               : launch_up<bf16, false>(x, W, wgu, E, idx, mid, ff, top, n_tok, act, in_wt, limit, st);
 }
 
-DK_EXPORT int dk_moe_down_rows(int dtype, const void* mid, const void* wd, const int* idx, const float* wt,
-                               const void* shared, const float* sgate, void* out, int W, int ff, int top, int n_tok,
+DK_EXPORT int dk_moe_down_rows(int dtype, const void* mid, const void* wd, int E, const int* idx, const float* wt,
+                               const void* shared, const float* sgate, const void* x, const float* in_wt, void* out, int W, int ff, int top, int n_tok,
                                cudaStream_t st) {
     const bool vec = (uintptr_t)wd % 16 == 0 && ff % (dtype == 0 ? 4 : 8) == 0;
     if (dtype == 0)
-        return vec ? launch_down<float, true>(mid, wd, idx, wt, shared, sgate, out, W, ff, top, n_tok, st)
-                   : launch_down<float, false>(mid, wd, idx, wt, shared, sgate, out, W, ff, top, n_tok, st);
-    return vec ? launch_down<bf16, true>(mid, wd, idx, wt, shared, sgate, out, W, ff, top, n_tok, st)
-               : launch_down<bf16, false>(mid, wd, idx, wt, shared, sgate, out, W, ff, top, n_tok, st);
+        return vec ? launch_down<float, true>(mid, wd, E, idx, wt, shared, sgate, x, in_wt, out, W, ff, top, n_tok, st)
+                   : launch_down<float, false>(mid, wd, E, idx, wt, shared, sgate, x, in_wt, out, W, ff, top, n_tok, st);
+    return vec ? launch_down<bf16, true>(mid, wd, E, idx, wt, shared, sgate, x, in_wt, out, W, ff, top, n_tok, st)
+               : launch_down<bf16, false>(mid, wd, E, idx, wt, shared, sgate, x, in_wt, out, W, ff, top, n_tok, st);
 }

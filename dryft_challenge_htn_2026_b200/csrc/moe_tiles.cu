@@ -6,6 +6,7 @@
 //   up:    mid[r] = act(W_gate[e] x_r) * (W_up[e] x_r)      rows gathered by token, both products in one pass
 //   down:  y[r]   = W_down[e] mid[r]
 //   sum:   out[t] = sum_j weight[t][j] * y[place of pair (t, j)] + gate[t] * shared[t]
+// Pairs of identity experts (numbers from E on) are in no tile; the sum takes the token's row itself for them.
 // A row's sums run over its own elements in a fixed order, so a result does not depend on which other pairs
 // share its tile. Grids are sized for the most tiles the pairs can make (pairs / 64 + experts); blocks
 // beyond the tiles that exist leave at once.
@@ -36,7 +37,7 @@ __device__ __forceinline__ void mt_commit() { asm volatile("cp.async.commit_grou
 template <int N> __device__ __forceinline__ void mt_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // One block. idx [P] = expert of every pair. Leaves perm [P] (pairs in expert order), inv [P] (a pair's place in
-// that order) and for every tile its expert, first place and row count in tiles [max_tiles][3] (rows 0: no tile).
+// that order, -1 for an identity expert's) and for every tile its expert, first place and row count in tiles [max_tiles][3] (rows 0: no tile).
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int* idx, int P, int E, int* perm, int* inv, int* tiles, int max_tiles) {
     __shared__ int cnt[256], off[257], tbase[257];
@@ -44,7 +45,10 @@ moe_sort_kernel(const int* idx, int P, int E, int* perm, int* inv, int* tiles, i
     pdl_launch_dependents();
     for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
     __syncthreads();
-    for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&cnt[idx[p]], 1);
+    for (int p = threadIdx.x; p < P; p += blockDim.x) {
+        const int e = idx[p];
+        if (e < E) atomicAdd(&cnt[e], 1);
+    }
     __syncthreads();
     if (threadIdx.x == 0) {
         off[0] = tbase[0] = 0;
@@ -66,6 +70,10 @@ moe_sort_kernel(const int* idx, int P, int E, int* perm, int* inv, int* tiles, i
     __syncthreads();
     for (int p = threadIdx.x; p < P; p += blockDim.x) {
         const int e = idx[p];
+        if (e >= E) {
+            inv[p] = -1;
+            continue;
+        }
         const int at = off[e] + atomicAdd(&cnt[e], 1);
         perm[at] = p;
         inv[p] = at;
@@ -192,15 +200,20 @@ moe_tile_product_kernel(const bf16* A, const bf16* __restrict__ B, const int* ti
         }
 }
 
-// out[t][c] = sum_j wt[t][j] * y[inv[t * top + j]][c] + sgate[t] * shared[t][c]
-__global__ void moe_sum_kernel(const bf16* y, const int* inv, const float* wt, const bf16* shared, const float* sgate, bf16* out,
-                               int W, int top) {
+// out[t][c] = sum_j wt[t][j] * y[inv[t * top + j]][c] + sgate[t] * shared[t][c]; a pair in no tile: wt[t][j] * x[t][c]
+// (in_wt: the pair's weight stood on the expert's input)
+__global__ void moe_sum_kernel(const bf16* y, const int* inv, const float* wt, const bf16* shared, const float* sgate, const bf16* x,
+                               const float* in_wt, bf16* out, int W, int top) {
     pdl_wait();
     pdl_launch_dependents();
     const size_t t = blockIdx.x;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float acc = 0.f;
-        for (int j = 0; j < top; j++) acc = fmaf(wt != nullptr ? wt[t * top + j] : 1.f, __bfloat162float(y[(size_t)inv[t * top + j] * W + c]), acc);
+        for (int j = 0; j < top; j++) {
+            const int at = inv[t * top + j];
+            const float* w = wt != nullptr ? wt : at < 0 ? in_wt : nullptr;
+            acc = fmaf(w != nullptr ? w[t * top + j] : 1.f, __bfloat162float(at < 0 ? x[t * W + c] : y[(size_t)at * W + c]), acc);
+        }
         if (shared != nullptr) acc = fmaf(sgate ? sgate[t] : 1.f, __bfloat162float(shared[t * W + c]), acc);
         out[t * W + c] = __float2bfloat16_rn(acc);
     }
@@ -239,8 +252,8 @@ DK_EXPORT int dk_moe_down_tiles(const void* mid, const void* wd, const int* tile
                      (const bf16*)wd, tiles, (const int*)nullptr, 1, (bf16*)y, W, ff, 0, (const float*)nullptr, 0.f);
 }
 
-DK_EXPORT int dk_moe_sum(const void* y, const int* inv, const float* wt, const void* shared, const float* sgate, void* out,
-                         int n_tok, int W, int top, cudaStream_t st) {
+DK_EXPORT int dk_moe_sum(const void* y, const int* inv, const float* wt, const void* shared, const float* sgate, const void* x,
+                         const float* in_wt, void* out, int n_tok, int W, int top, cudaStream_t st) {
     return dk_launch(moe_sum_kernel, dim3(n_tok), dim3(W >= 1024 ? 256 : 128), 0, st, (const bf16*)y, inv, wt, (const bf16*)shared,
-                     sgate, (bf16*)out, W, top);
+                     sgate, (const bf16*)x, in_wt, (bf16*)out, W, top);
 }

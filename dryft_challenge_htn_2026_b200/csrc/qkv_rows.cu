@@ -4,7 +4,8 @@
 //     place in the paged stores. q and k: an RMS norm, with a weight or without, over all heads at once before the
 //     rotation (norm_mode 3, weights of the whole projection's size), per head before it (1) or per head behind it (2);
 //     a rotation of the first rot_dims coordinates, halves (i with i + rot_dims / 2) or neighbouring pairs (2i with 2i + 1),
-//     by tables [positions, rot_dims / 2]. v: a rotation over the whole value head by tables of its own.
+//     by tables [positions, rot_dims / 2]. v: a rotation over the whole value head by tables of its own. Rows may also be
+//     [q heads | k heads]: the values are then the keys as projected, before norm and rotation.
 //   * turn_back_gate: per head the attention's output turned back by the token's position (the same tables, the sine
 //     negated), times sigmoid of one gate number per head, times a constant.
 // Norms, rotations and gates are float32 whatever the storage type. Rows with position < 0 are padding.
@@ -127,7 +128,7 @@ qkv_rows_kernel(const T* proj, long long ld, T* q_out, long long ldq, int norm_m
                 const float* __restrict__ kn, float eps, const float* __restrict__ cosv, const float* __restrict__ sinv,
                 int rot_dims, int pairs, const float* __restrict__ vcos, const float* __restrict__ vsin, int v_pairs,
                 const int* row_pos, const int* row_seq, int nh, int nkv, int hd, int hdv, T* k_store, T* v_store,
-                const int* page_table, int pt_stride, int vec) {
+                const int* page_table, int pt_stride, int kv_same, int vec) {
     __shared__ float ys_all[QR_WARPS][128 * NI];
     __shared__ float2 sums[QR_WARPS];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
@@ -141,7 +142,7 @@ qkv_rows_kernel(const T* proj, long long ld, T* q_out, long long ldq, int norm_m
         for (int n = 0; n < HPW; n++) {
             const int head = head0 + n * gridDim.y * QR_WARPS;
             const bool is_v = head >= nh + nkv;
-            const T* src = row + (is_v ? nq + nk + (head - nh - nkv) * hdv : head * hd);
+            const T* src = row + (is_v ? nq + (kv_same ? 0 : nk) + (head - nh - nkv) * hdv : head * hd);
 #pragma unroll
             for (int i = 0; i < NI; i++) ld_four<T>(src, 4 * lane + 128 * i, head >= heads ? 0 : is_v ? hdv : hd, vec, y[n][i]);
         }
@@ -288,9 +289,9 @@ DK_EXPORT int dk_qkv_rows(int dtype, const void* proj, long long ld, void* q_out
                           const float* kn, float eps, const float* cosv, const float* sinv, int rot_dims, int pairs,
                           const float* vcos, const float* vsin, int v_pairs, const int* row_pos, const int* row_seq, int n_tok,
                           int nh, int nkv, int hd, int hdv, void* k_store, void* v_store, const int* page_table, int pt_stride,
-                          cudaStream_t st) {
+                          int kv_same, cudaStream_t st) {
     if (hd < 1 || hd > 256 || hdv < 1 || hdv > 256 || rot_dims > hd || rot_dims % 2 || (vcos != nullptr && hdv % 2) ||
-        norm_mode < 0 || norm_mode > 3)
+        norm_mode < 0 || norm_mode > 3 || (kv_same && hd != hdv))
         return (int)cudaErrorInvalidValue;
     const int esz = dtype == 0 ? 4 : 2;
     const int vec = hd % 4 == 0 && hdv % 4 == 0 && ld % 4 == 0 && ldq % 4 == 0 &&
@@ -305,7 +306,7 @@ DK_EXPORT int dk_qkv_rows(int dtype, const void* proj, long long ld, void* q_out
 #define QR_LAUNCH(T, NI, HPW)                                                                                                \
     return dk_launch(qkv_rows_kernel<T, NI, HPW>, grid, block, 0, st, (const T*)proj, ld, (T*)q_out, ldq, norm_mode, qn, kn, eps, \
                      cosv, sinv, rot_dims, pairs, vcos, vsin, v_pairs, row_pos, row_seq, nh, nkv, hd, hdv, (T*)k_store,      \
-                     (T*)v_store, page_table, pt_stride, vec)
+                     (T*)v_store, page_table, pt_stride, kv_same, vec)
     const bool small = hd <= 128 && hdv <= 128;
     if (dtype == 0) {
         if (small) QR_LAUNCH(float, 1, 3);

@@ -6,7 +6,8 @@
 //   * sublayer_add      : h_out = h + norm(d), and a = that row in the storage type, or its next norm. d is a sublayer's
 //                         output (a tensor or split-K partial sums), or a scaled sum of two of them, each over its own root
 //                         mean square times a weight first. norm is a layer norm (mean taken off) or an RMS norm, with a
-//                         weight, or none. With ``rows`` the kernel gathers and leaves h alone. It may also put the stream as
+//                         weight and, where given, a bias, or none. Without an h the stream starts anew from a vector (null:
+//                         zero), the same for every row. With ``rows`` the kernel gathers and leaves h alone. It may also put the stream as
 //                         it stood BEFORE the sum into the shift's state at every sequence's last row: that is the vector the
 //                         mixer in front of it has read, and by now every reader of the old state is done.
 //   * sublayer_add_shift: the same sum, then a = x + (x_prev - x) * share with x_prev the row of the token before (the
@@ -25,6 +26,7 @@ template <typename T> struct Source {
 };
 struct NormArgs {
     const float* w;          // null: no norm
+    const float* b;          // null: no bias
     float eps;
     int center;              // 1: layer norm, 0: RMS norm
 };
@@ -126,6 +128,11 @@ __device__ __forceinline__ void norm_row(float (&d)[NV][4], const NormArgs& n, i
         ld_cols(n.w, (threadIdx.x + q * blockDim.x) * 4, H, vec, w);
 #pragma unroll
         for (int k = 0; k < 4; k++) d[q][k] *= rs * w[k];
+        if (n.b) {
+            ld_cols(n.b, (threadIdx.x + q * blockDim.x) * 4, H, vec, w);
+#pragma unroll
+            for (int k = 0; k < 4; k++) d[q][k] += w[k];
+        }
     }
 }
 
@@ -150,9 +157,13 @@ __device__ __forceinline__ void load_source(float (&d)[NV][4], const Source<T>& 
 // v <- h[row] + norm(delta[row]): first the loads, which wait for nothing, ...
 template <typename T, int NV, bool TWO>
 __device__ __forceinline__ void load_row(float (&v)[NV][4], float (&d)[NV][4], float (&e)[TWO ? NV : 1][4], const float* h, size_t row,
-                                         const AddArgs<T>& a, int H, bool vec) {
+                                         const AddArgs<T>& a, int H, bool vec, const float* base = nullptr) {
+    const float* from = h ? h + row * H : base;          // the stream, or the vector it starts anew from
 #pragma unroll
-    for (int q = 0; q < NV; q++) ld_cols(h + row * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
+    for (int q = 0; q < NV; q++) {
+        if (from) ld_cols(from, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
+        else v[q][0] = v[q][1] = v[q][2] = v[q][3] = 0.f;
+    }
     if (a.s0.x || a.s0.parts) load_source<T, NV>(d, a.s0, row, H, vec);
     if constexpr (TWO) load_source<T, NV>(e, a.s1, row, H, vec);
 }
@@ -195,7 +206,7 @@ __device__ __forceinline__ void sum_row(float (&v)[NV][4], float (&d)[NV][4], fl
 
 template <typename T, int NV, bool TWO, int MAXT>
 __global__ void __launch_bounds__(MAXT)
-sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const int* rows, NormArgs next, T* a, float* save,
+sublayer_add_kernel(const float* h, const float* base, float* h_out, const AddArgs<T> args, const int* rows, NormArgs next, T* a, long long lda, float* save,
                     const int* row_pos, const int* row_seq, const int* cu_q, const int* seq_slot, int H, int vec) {
     __shared__ float2 red[2][32];
     BlockSums sums{red, 0};
@@ -203,7 +214,7 @@ sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const i
     pdl_launch_dependents();
     const size_t out_row = blockIdx.x, row = rows ? (size_t)rows[out_row] : out_row;
     float v[NV][4], d[NV][4], e[TWO ? NV : 1][4];
-    load_row<T, NV, TWO>(v, d, e, h, row, args, H, vec);
+    load_row<T, NV, TWO>(v, d, e, h, row, args, H, vec, base);
     if (save != nullptr && row_pos[row] >= 0) {
         const int s = row_seq[row];
         if (cu_q == nullptr || (int)row + 1 == cu_q[s + 1]) {
@@ -220,7 +231,7 @@ sublayer_add_kernel(const float* h, float* h_out, const AddArgs<T> args, const i
     if (a == nullptr) return;
     if (next.w) norm_row<NV>(v, next, H, vec, sums);
 #pragma unroll
-    for (int q = 0; q < NV; q++) st_cols(a + out_row * H, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
+    for (int q = 0; q < NV; q++) st_cols(a + out_row * lda, (threadIdx.x + q * blockDim.x) * 4, H, vec, v[q]);
 }
 
 template <typename T, int NV, bool TWO, int MAXT>
@@ -326,35 +337,35 @@ static inline int stream_threads(int H, int n_rows) {
 template <typename T>
 static AddArgs<T> make_add(const void* x0, const float* parts0, int n0, long long stride0, const float* w0, const void* x1,
                            const float* parts1, int n1, long long stride1, const float* w1, float pre_eps, float pre_scale,
-                           const float* norm_w, float eps, int center) {
+                           const float* norm_w, const float* norm_b, float eps, int center) {
     AddArgs<T> a;
     a.s0 = {(const T*)x0, parts0, n0, (size_t)stride0, w0};
     a.s1 = {(const T*)x1, parts1, n1, (size_t)stride1, w1};
     a.pre_eps = pre_eps, a.pre_scale = pre_scale;
-    a.norm = {norm_w, eps, center};
+    a.norm = {norm_w, norm_b, eps, center};
     return a;
 }
 
 #define ADD_PARAMS const void *x0, const float *parts0, int n0, long long stride0, const float *w0, const void *x1,          \
                    const float *parts1, int n1, long long stride1, const float *w1, float pre_eps, float pre_scale,          \
-                   const float *norm_w, float eps, int center
-#define ADD_NAMES x0, parts0, n0, stride0, w0, x1, parts1, n1, stride1, w1, pre_eps, pre_scale, norm_w, eps, center
+                   const float *norm_w, const float *norm_b, float eps, int center
+#define ADD_NAMES x0, parts0, n0, stride0, w0, x1, parts1, n1, stride1, w1, pre_eps, pre_scale, norm_w, norm_b, eps, center
 // four columns at a time where rows, partial sums and every pointer sit on 16-byte boundaries
 #define ADD_VEC (H % 4 == 0 && stride0 % 4 == 0 && stride1 % 4 == 0 &&                                                        \
                  (((uintptr_t)h | (uintptr_t)h_out | (uintptr_t)x0 | (uintptr_t)parts0 | (uintptr_t)w0 | (uintptr_t)x1 |      \
-                   (uintptr_t)parts1 | (uintptr_t)w1 | (uintptr_t)norm_w | (uintptr_t)a) % 16 == 0))
+                   (uintptr_t)parts1 | (uintptr_t)w1 | (uintptr_t)norm_w | (uintptr_t)norm_b | (uintptr_t)a) % 16 == 0))
 
-DK_EXPORT int dk_sublayer_add(int dtype, const float* h, float* h_out, ADD_PARAMS, const int* rows, const float* next_w,
-                              float next_eps, int next_center, void* a, float* save, const int* row_pos, const int* row_seq,
+DK_EXPORT int dk_sublayer_add(int dtype, const float* h, const float* base, float* h_out, ADD_PARAMS, const int* rows, const float* next_w,
+                              const float* next_b, float next_eps, int next_center, void* a, long long lda, float* save, const int* row_pos, const int* row_seq,
                               const int* cu_q, const int* seq_slot, int n_rows, int H, cudaStream_t st) {
     if (H < 1 || H > 16384) return (int)cudaErrorInvalidValue;
     const int threads = stream_threads(H, n_rows), nv = ((H + 3) / 4 + threads - 1) / threads;
-    const int vec = ADD_VEC && ((uintptr_t)next_w | (uintptr_t)save) % 16 == 0;
-    const NormArgs next = {next_w, next_eps, next_center};
+    const int vec = ADD_VEC && lda % 4 == 0 && ((uintptr_t)next_w | (uintptr_t)next_b | (uintptr_t)base | (uintptr_t)save) % 16 == 0;
+    const NormArgs next = {next_w, next_b, next_eps, next_center};
     const bool two = x1 != nullptr || parts1 != nullptr;
 #define ADD_GO(NV, TWO, MAXT)                                                                                                       \
-    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_kernel<T, NV, TWO, MAXT>, dim3(n_rows), dim3(threads), 0, st, h, h_out,     \
-                                            make_add<T>(ADD_NAMES), rows, next, (T*)a, save, row_pos, row_seq, cu_q, seq_slot, \
+    STREAM_DISPATCH(dtype, return dk_launch(sublayer_add_kernel<T, NV, TWO, MAXT>, dim3(n_rows), dim3(threads), 0, st, h, base, h_out,     \
+                                            make_add<T>(ADD_NAMES), rows, next, (T*)a, lda, save, row_pos, row_seq, cu_q, seq_slot, \
                                             H, vec))
 #define ADD_LAUNCH(NV, MAXT)                                                                                                         \
     if (nv <= NV && threads <= MAXT) {                                                                  \

@@ -8,8 +8,8 @@ from ..cache.requests import StateRequest
 from ..csrc import api
 from ..parts import ParamDecl, Runtime, build_part
 from ..parts.block import add_norm
-from ..parts.linear import STORE_F32, linear
-from ..parts.norm import RMSNorm
+from ..parts.linear import STORE_F32, linear, linear_partial
+from ..parts.norm import NormedDelta, RMSNorm, StreamReset, norm_args
 
 
 class CausalLM:
@@ -50,7 +50,14 @@ class CausalLM:
         for e in spec.schedule:
             if e.add_row is not None and e.add_row[0] not in names:
                 raise ValueError(f"schedule adds a row of {e.add_row[0]!r}, which is not a table of the model")
+        self.matrices = {}       # the model's own learned matrices (ModelSpec.matrices), by name
+        wide = {n for n, shape in spec.matrices if tuple(shape) == (spec.hidden_size, 2 * spec.hidden_size)}
+        for e in spec.schedule:
+            if e.take_in is not None and (e.take_in not in wide or e.add_embedding):
+                raise ValueError(f"a run takes the embedding in by {e.take_in!r}, which is not a matrix [hidden, 2 hidden] of the "
+                                 "model, or adds it as well")
         self._keeps_embedding = any(e.add_embedding for e in spec.schedule)
+        self._takes_in = any(e.take_in is not None for e in spec.schedule)
         # index arrays the parts' kernels want built for every step (engine.batch.build_context), once per key
         self.step_plans = list({p.key: p for b in self.blocks for p in b.step_plans()}.values())
         self.prepared = 0        # positions the parts' tables reach
@@ -71,6 +78,8 @@ class CausalLM:
             out[s.final_norm_prefix + p.name] = p
         for name, shape in s.tables:
             out[name] = ParamDecl(name, tuple(shape), "matrix", keep_float32=True)
+        for name, shape in s.matrices:
+            out[name] = ParamDecl(name, tuple(shape), "matrix")
         if not tied:
             out[s.head_name] = ParamDecl(s.head_name, (s.vocab_size, s.hidden_size), "matrix")
         return out
@@ -83,6 +92,7 @@ class CausalLM:
         if s.embed_bigram is not None:
             self.bigram = tensors.pop(s.embed_bigram.tensor).contiguous()
         self.tables = {name: tensors.pop(name).to(torch.float32).contiguous() for name, _ in s.tables}
+        self.matrices = {name: tensors.pop(name).contiguous() for name, _ in s.matrices}
         for ls, blk in zip(s.layers, self.blocks):
             n = len(ls.prefix)
             blk.bind({k[n:]: tensors.pop(k) for k in [k for k in tensors if k.startswith(ls.prefix)]})
@@ -109,9 +119,20 @@ class CausalLM:
         total = self.head.numel() * self.head.element_size()
         for e in self.spec.schedule:
             total += sum(w.numel() * w.element_size() for w in self.blocks[e.layer].step_weights())
+            if e.take_in is not None:
+                total += self.matrices[e.take_in].numel() * self.matrices[e.take_in].element_size()
         return total
 
     # -- one step ----------------------------------------------------------------------------
+    def _take_in(self, h, pending, both, matrix, row):
+        """The stream x (``h`` with what is still ``pending``) becomes M [x; x0] (+ ``row``): ``both`` [rows, 2 hidden] holds x0
+        in its second half, in the storage type, and gets x in its first. -> the ``StreamReset`` the next block starts from."""
+        norm = None
+        if isinstance(pending, NormedDelta):
+            pending, norm = pending.delta, norm_args(pending.norm)
+        api.sublayer_add(h, pending, norm, both[:, :self.spec.hidden_size])
+        return StreamReset(linear_partial(both, matrix), row)
+
     def forward(self, ctx, cache, tap=None):
         """``tap(k, h)``: called after the k-th schedule entry with the residual stream as it then
         stands (that entry's feed-forward output added in): for dumps that look for the layer where
@@ -121,11 +142,13 @@ class CausalLM:
         a = torch.empty((ctx.n_tok, s.hidden_size), dtype=rt.dtype, device=rt.device)
         first = self.blocks[s.schedule[0].layer]
         # the embedding kernel computes RMSNorm and nothing else, and only of the embedding as it leaves the kernel
-        fused = isinstance(getattr(first, "norm_in", None), RMSNorm) and not (s.schedule[0].add_embedding or s.schedule[0].add_row)
+        fused = isinstance(getattr(first, "norm_in", None), RMSNorm) and not (
+            s.schedule[0].add_embedding or s.schedule[0].add_row or s.schedule[0].take_in)
         norm_w, eps = (first.norm_in.weight, first.norm_in.spec.eps) if fused else (None, 0.0)
         ctx.carry = {}           # what one layer of the step leaves for later ones (e.g. values that layers share)
         ctx.stream_copy = None   # the stream in the storage type, where a kernel has left it (blocks with the norm after the sum)
-        plain = getattr(first, "reads_stream", False) and not (s.schedule[0].add_embedding or s.schedule[0].add_row)
+        plain = getattr(first, "reads_stream", False) and not (
+            s.schedule[0].add_embedding or s.schedule[0].add_row or s.schedule[0].take_in)
         ctx.stream = None        # the stream, where a block has written it to another buffer than the one it was given
         if self.bigram is not None:
             b = s.embed_bigram
@@ -140,9 +163,17 @@ class CausalLM:
             api.embed_position_rmsnorm(ctx.tok, self.embed, s.embed_scale, ctx.row_pos,
                                        self.position.inv_freq if self.position is not None else None, norm_w, eps, h, a)
         e0 = h.clone() if self._keeps_embedding else None     # the embedding's output, for the runs that take it in again
+        both = None
+        if self._takes_in:       # [x | x0] for the runs that take the embedding in by a matrix: x0 stays in its half
+            both = torch.empty((ctx.n_tok, 2 * s.hidden_size), dtype=rt.dtype, device=rt.device)
+            api.sublayer_add(h, None, None, both[:, s.hidden_size:])
         pending = None
         for i, e in enumerate(s.schedule):
-            if e.add_embedding or e.add_row is not None:
+            if e.take_in is not None:
+                pending = self._take_in(h, pending, both, self.matrices[e.take_in],
+                                        self.tables[e.add_row[0]][e.add_row[1]] if e.add_row is not None else None)
+                ctx.stream_copy = None
+            elif e.add_embedding or e.add_row is not None:
                 api.stream_add(h, e0 if e.add_embedding else None,
                                self.tables[e.add_row[0]][e.add_row[1]] if e.add_row is not None else None)
                 ctx.stream_copy = None

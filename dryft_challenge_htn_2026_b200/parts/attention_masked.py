@@ -4,7 +4,7 @@ switched on by its specification; key and value heads may differ in size.
 
 forward = one fused projection [q; k; v; gate] -> (where the specification asks: a short causal convolution
 over time on q, k and v with a per-sequence state, a norm per q and k head, a rotation of the heads' first
-coordinates; one kernel; or q and k normed as whole projections, rotated by pairs, values turned by their position: another) -> k and v into the cache -> attention over the cache with the gate in its epilogue
+coordinates; one kernel; or q and k normed as whole projections, rotated by pairs, values turned by their position or the keys as projected: another) -> k and v into the cache -> attention over the cache with the gate in its epilogue
 (a kernel behind it where turned values are turned back or each head has one gate) -> output projection. Further options of the scores: a cap, first tokens that the window keeps, a sink fixed
 at zero. Kernels: bfloat16 prompts with equal head sizes of 64
 or 128 on tcgen05 tensor cores, other head sizes in steps of 16 on mma.sync, single tokens by a kernel of
@@ -36,11 +36,15 @@ class MaskedAttention(Part):
             raise ValueError(f"values of {s.v_head_dim} numbers cannot be the start of key rows of {s.head_dim}")
         self.n_q, self.n_k = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
         self.n_v, self.n_mid = s.num_kv_heads * s.v_head_dim, s.num_heads * s.v_head_dim
+        if s.keys_as_values:         # the values are the k columns of the projection
+            if s.v_head_dim != s.head_dim:
+                raise ValueError(f"keys of {s.head_dim} numbers are not values of {s.v_head_dim}")
+            self.n_v = 0
         if s.head_gate and s.output_gate:
             raise ValueError("a gate per head and a gate per coordinate exclude each other")
         self.n_gate = self.n_mid if s.output_gate else s.num_heads if s.head_gate else 0
         self.n_in = self.n_q + self.n_k + self.n_v + self.n_gate
-        if s.head_gate:      # a few gate rows behind q, k, v: filled up with zero rows, so that rows of the product stay aligned
+        if s.head_gate or s.keys_as_values:      # filled up with zero rows, so that rows of the product stay aligned
             self.n_in = (self.n_in + 7) // 8 * 8
         self.r1 = self.r2 = self.sink = None
         if s.unit_sink:
@@ -70,9 +74,9 @@ class MaskedAttention(Part):
             raise ValueError(f"a query temperature every {s.q_temp[1]} positions")
         # q and k normed as wholes, a rotation by pairs, values that turn: the row kernel without convolution and biases
         self.value_position = build_part(s.value_position, rt) if s.value_position is not None else None
-        self.row_kernel = self.value_position is not None or s.qk_norm_whole or getattr(self.position, "pairs", False)
+        self.row_kernel = self.value_position is not None or s.qk_norm_whole or s.keys_as_values or getattr(self.position, "pairs", False)
         if self.row_kernel and (s.conv_taps not in (None, 1) or s.bias or s.q_temp is not None or s.value_mix is not None or s.talk):
-            raise ValueError("rotation by pairs, a norm of the whole projection and turning values go without a convolution, "
+            raise ValueError("rotation by pairs, a norm of the whole projection, turning values and keys as values go without a convolution, "
                              "biases, a query temperature, blended values and mixed head scores")
         if self.value_position is not None and self.value_position.spec.dim != s.v_head_dim:
             raise ValueError(f"values of {s.v_head_dim} turned over {self.value_position.spec.dim} coordinates")
@@ -109,8 +113,10 @@ class MaskedAttention(Part):
 
     def param_decls(self):
         s = self.spec
-        d = [ParamDecl("q", (self.n_q, s.hidden_size)), ParamDecl("k", (self.n_k, s.hidden_size)),
-             ParamDecl("v", (self.n_v, s.hidden_size)), ParamDecl("o", (s.hidden_size, self.n_mid))]
+        d = [ParamDecl("q", (self.n_q, s.hidden_size)), ParamDecl("k", (self.n_k, s.hidden_size))]
+        if not s.keys_as_values:
+            d.append(ParamDecl("v", (self.n_v, s.hidden_size)))
+        d.append(ParamDecl("o", (s.hidden_size, self.n_mid)))
         if self.n_gate:
             d.append(ParamDecl("g", (self.n_gate, s.hidden_size)))
         if s.distance_bias:
@@ -135,7 +141,7 @@ class MaskedAttention(Part):
         return d
 
     def bind(self, tensors):
-        rows = [tensors.pop("q"), tensors.pop("k"), tensors.pop("v")]
+        rows = [tensors.pop("q"), tensors.pop("k")] + ([] if self.spec.keys_as_values else [tensors.pop("v")])
         if self.n_gate:
             rows.append(tensors.pop("g"))
         fill = self.n_in - sum(w.shape[0] for w in rows)
@@ -193,7 +199,7 @@ class MaskedAttention(Part):
         api.qkv_rows(proj[:, :self.n_qkv], out, mode, self.q_norm_w, self.k_norm_w, self.qk_norm.eps if self.qk_norm is not None else 0.0,
                      self._rotation(ctx, self.position), self._rotation(ctx, self.value_position), ctx.row_pos, ctx.row_seq,
                      s.num_heads, s.num_kv_heads, s.head_dim, s.v_head_dim, kv.k if writes else None, kv.v if writes else None,
-                     ctx.tables[kv.group] if writes else None)
+                     ctx.tables[kv.group] if writes else None, keys_as_values=s.keys_as_values)
         return out
 
     def prepared_rows(self, ctx, views, proj, writes=True):

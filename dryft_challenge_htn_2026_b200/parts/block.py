@@ -12,7 +12,7 @@ from ..cache.requests import StateRequest
 from ..config.specs import LayerSpec, OutputNormLayerSpec, PostNormLayerSpec, SandwichLayerSpec
 from ..csrc import api
 from .base import ParamDecl, Part, build_part, register_part
-from .norm import NormedDelta, RMSNorm, norm_args
+from .norm import NormedDelta, RMSNorm, StreamReset, norm_args
 
 
 class PreNormBlock(Part):
@@ -63,6 +63,9 @@ class PreNormBlock(Part):
 
 def add_norm(norm, h, delta, dtype, rows=None):
     """h += delta, then norm(h) (of the rows ``rows`` only, leaving h alone, when given)."""
+    if isinstance(delta, StreamReset) and not getattr(norm, "takes_reset", False):
+        delta.write(h)
+        delta = None
     if isinstance(delta, NormedDelta) and not isinstance(norm, RMSNorm) and not getattr(norm, "takes_normed", False):
         raise TypeError(f"{type(norm).__name__} cannot follow a sublayer whose output has a norm of its own")
     if isinstance(delta, api.Partial) and not getattr(norm, "takes_partial", False):
@@ -102,6 +105,9 @@ class PostNormBlock(Part):
 
     def forward(self, ctx, h, pending, views, writes=True, a=None):
         dtype = self.rt.dtype
+        if isinstance(pending, StreamReset):
+            pending.write(h)
+            pending = ctx.stream_copy = None
         if pending is not None:          # a block before this one left its output to be added
             if isinstance(pending, NormedDelta):
                 pending = pending.to_float32()
@@ -141,8 +147,24 @@ class SandwichBlock(PreNormBlock):
         self.feed_forward = build_part(spec.feed_forward, rt) if has_ff else None
         self.norm_ff_out = build_part(spec.norm_ff_out, rt) if has_ff else None
         for n in (self.norm_in, self.norm_mix_out, self.norm_post, self.norm_ff_out):
-            if n is not None and not isinstance(n, RMSNorm):
-                raise TypeError(f"{type(n).__name__}: the norms around a sublayer run on the RMS norm's kernels")
+            if n is not None and not isinstance(n, RMSNorm) and not getattr(n, "takes_normed", False):
+                raise TypeError(f"{type(n).__name__}: the norms around a sublayer run on the RMS norm's or the layer norm's kernels")
+        inner = [n for n in (self.norm_in, self.norm_post) if n is not None]
+        outer = [n for n in (self.norm_mix_out, self.norm_ff_out) if n is not None]
+        if any(isinstance(n, RMSNorm) for n in inner) and not all(isinstance(n, RMSNorm) for n in outer):
+            raise TypeError("the RMS norm's kernels take RMS norms on the sublayers' outputs")
+
+    def _scales(self):
+        """(name, norm) of the vectors that multiply what the sublayers add."""
+        return [(name, n) for name, n in zip(self.spec.layer_scale or (), (self.norm_mix_out, self.norm_ff_out)) if n is not None]
+
+    def param_decls(self):
+        return PreNormBlock.param_decls(self) + [ParamDecl(name, (n.spec.dim,), init="norm", keep_float32=True) for name, n in self._scales()]
+
+    def bind(self, tensors):
+        PreNormBlock.bind(self, tensors)
+        for name, n in self._scales():       # into the output norm's own weight and bias
+            n.scale_output(tensors.pop(name).to(torch.float32))
 
     def forward(self, ctx, h, pending, views, writes=True, a=None):
         if a is None:
@@ -191,6 +213,9 @@ class OutputNormBlock(PreNormBlock):
 
     def forward(self, ctx, h, pending, views, writes=True, a=None):
         dtype = self.rt.dtype
+        if isinstance(pending, StreamReset):
+            pending.write(h)
+            pending = None
         delta, norm = (pending.delta, norm_args(pending.norm)) if isinstance(pending, NormedDelta) else (pending, None)
         a = torch.empty(h.shape, dtype=dtype, device=h.device)
         save = None

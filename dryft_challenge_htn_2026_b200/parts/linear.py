@@ -20,7 +20,7 @@ def linear(x, w, mode=STORE, allow_partial=False, act=(0.0, 0.0)):
     (alpha_pos, alpha_neg), in the product's epilogue wherever the product is this library's (after
     the library's product a row kernel applies it). ``allow_partial``: the caller can take
     ``csrc.api.Partial`` (split-K partial sums, added up by the kernel that consumes them) instead
-    of a tensor."""
+    of a tensor (with STORE_F32 too: partial sums are float32)."""
     M, K = x.shape
     N = w.shape[0] // 2 if mode == SILU else w.shape[0]
     if x.dtype == torch.float32:
@@ -50,7 +50,8 @@ def linear(x, w, mode=STORE, allow_partial=False, act=(0.0, 0.0)):
     if M <= api.TC_SKINNY_MAX_ROWS:
         # a decode step of up to 128 rows: weights streamed once by TMA, one 128-row tile of x,
         # K in slices so that the few weight tiles still cover the SMs
-        return api.gemm_tc(x, w, mode, None, api.skinny_tc_plan(M, N, K, mode, allow_partial), act)
+        plan = api.skinny_tc_plan(M, N, K, STORE if mode == STORE_F32 and allow_partial else mode, allow_partial)
+        return api.gemm_tc(x, w, STORE if mode == STORE_F32 and plan[1] > 1 else mode, None, plan, act)
     if mode == STORE_F32:
         return torch.mm(x, w.t(), out_dtype=torch.float32)
     if mode == SILU:
@@ -61,3 +62,9 @@ def linear(x, w, mode=STORE, allow_partial=False, act=(0.0, 0.0)):
     if mode == XIELU:
         api.xielu(out, out, act[0], act[1])
     return out
+
+
+def linear_partial(x, w):
+    """x . w^T in float32 as a ``csrc.api.Partial`` (of one slice or more), for the kernels that put it into the stream."""
+    y = linear(x, w, STORE_F32, allow_partial=True)
+    return y if isinstance(y, api.Partial) else api.Partial(y.unsqueeze(0))

@@ -1,6 +1,6 @@
 """Mixture of experts: a router in float32, routed gated feed-forwards, an optional shared expert with a gate.
 
-forward = router kernel (sigmoid scores, choice by score + correction among the best groups, weights from the
+forward = router kernel (sigmoid or softmax scores, choice by score + correction among the best groups, weights from the
 scores alone; also the shared expert's gate) -> the chosen experts' gate/up products with the activation ->
 their down products, weighted and summed per token, plus gate * shared expert. Steps of many tokens in bfloat16
 sort the (token, expert) pairs by expert on the device and run tiles of one expert on the tensor cores; single
@@ -23,11 +23,14 @@ class RoutedMLP(Part):
         s = spec
         if s.activation not in _ACTS:
             raise ValueError(f"activation {s.activation!r} is not implemented ({sorted(_ACTS)})")
-        if s.num_experts > api.MOE_MAX_EXPERTS or s.num_experts % s.groups or not 1 <= s.keep_groups <= s.groups or \
-                not 1 <= s.top <= min(s.num_experts, 32):
-            raise ValueError(f"{s.num_experts} experts in {s.groups} groups, {s.keep_groups} kept, {s.top} chosen")
-        if s.top > s.keep_groups * (s.num_experts // s.groups):
-            raise ValueError(f"{s.top} experts cannot be chosen from {s.keep_groups} groups of {s.num_experts // s.groups}")
+        self.n_out = s.num_experts + s.identity          # router outputs: the experts, then the identity experts
+        if s.identity < 0 or self.n_out > api.MOE_MAX_EXPERTS or self.n_out % s.groups or not 1 <= s.keep_groups <= s.groups or \
+                not 1 <= s.top <= min(self.n_out, 32):
+            raise ValueError(f"{s.num_experts} + {s.identity} experts in {s.groups} groups, {s.keep_groups} kept, {s.top} chosen")
+        if s.top > s.keep_groups * (self.n_out // s.groups):
+            raise ValueError(f"{s.top} experts cannot be chosen from {s.keep_groups} groups of {self.n_out // s.groups}")
+        if s.scores not in ("sigmoid", "softmax") or s.group_top not in (1, 2):
+            raise ValueError(f"router scores {s.scores!r} (sigmoid, softmax), groups scored by {s.group_top} (1 or 2)")
         if s.shared_ff is not None and s.activation not in ("silu", "clamped"):
             raise ValueError("the shared expert runs with SiLU or the clamped gate only")
         if s.activation == "clamped" and (s.limit is None or not s.limit > 0 or
@@ -40,9 +43,9 @@ class RoutedMLP(Part):
         for e in range(s.num_experts):
             d += [ParamDecl(f"e{e}.gate", (s.expert_ff, s.hidden_size)), ParamDecl(f"e{e}.up", (s.expert_ff, s.hidden_size)),
                   ParamDecl(f"e{e}.down", (s.hidden_size, s.expert_ff))]
-        d.append(ParamDecl("router", (s.num_experts, s.hidden_size), init="wide", keep_float32=True))
+        d.append(ParamDecl("router", (self.n_out, s.hidden_size), init="wide", keep_float32=True))
         if s.correction:
-            d.append(ParamDecl("correction", (s.num_experts,), init="around_zero", keep_float32=True))
+            d.append(ParamDecl("correction", (self.n_out,), init="around_zero", keep_float32=True))
         if s.shared_ff is not None:
             d += [ParamDecl("shared.gate", (s.shared_ff, s.hidden_size)), ParamDecl("shared.up", (s.shared_ff, s.hidden_size)),
                   ParamDecl("shared.down", (s.hidden_size, s.shared_ff))]
@@ -79,7 +82,7 @@ class RoutedMLP(Part):
         wt = torch.empty((T, s.top), dtype=torch.float32, device=dev)
         sgate = torch.empty((T,), dtype=torch.float32, device=dev) if self.w_shared_gate is not None else None
         api.moe_route(a, self.w_router, self.correction, self.w_shared_gate, s.top, s.groups, s.keep_groups, s.route_scale,
-                      idx, wt, sgate, renorm=s.renorm)
+                      idx, wt, sgate, renorm=s.renorm, softmax=s.scores == "softmax", group_top=s.group_top)
         shared = None
         if s.shared_ff is not None and s.activation == "clamped":      # the clamped gate in the product's epilogue
             shared = linear(linear(a, self.w_shared_gu, SILU, act=api.gate_clamped(s.shared_limit)), self.w_shared_down)
@@ -97,7 +100,7 @@ class RoutedMLP(Part):
         # few tokens (a pair reads its expert's matrices once), float32, or sizes the tiles do not take
         mid = torch.empty((T * s.top, s.expert_ff), dtype=self.rt.dtype, device=dev)
         api.moe_up_rows(a, self.w_gate_up, idx, mid, _ACTS[s.activation], in_wt=w_in, limit=limit)
-        api.moe_down_rows(mid, self.w_down, idx, w_out, shared, sgate, out)
+        api.moe_down_rows(mid, self.w_down, idx, w_out, shared, sgate, out, x=a if s.identity else None, in_wt=w_in)
         return out
 
 

@@ -20,7 +20,22 @@ class NormedDelta:
             self.delta.ws.sum(0) if isinstance(self.delta, api.Partial) else self.delta.to(torch.float32)
         if isinstance(self.norm, LayerNorm):
             d = d - d.mean(-1, keepdim=True)
-        return d * torch.rsqrt((d * d).mean(-1, keepdim=True) + self.norm.spec.eps) * self.norm.weight
+        d = d * torch.rsqrt((d * d).mean(-1, keepdim=True) + self.norm.spec.eps) * self.norm.weight
+        bias = getattr(self.norm, "bias", None)
+        return d if bias is None else d + bias
+
+
+class StreamReset:
+    """What comes to a block in place of the output of the one before where the stream starts anew: the stream becomes
+    ``delta`` (a ``csrc.api.Partial``) plus the vector ``base`` (or none), whatever it was. A norm that says ``takes_reset``
+    does that and the norm in one kernel."""
+
+    def __init__(self, delta, base=None):
+        self.delta, self.base = delta, base
+
+    def write(self, h):
+        """The plain form: the new stream into ``h``."""
+        api.sublayer_add(None, self.delta, None, None, h_out=h, base=self.base)
 
 
 class RMSNorm(Part):
@@ -32,6 +47,10 @@ class RMSNorm(Part):
 
     def bind(self, tensors):
         self.weight = tensors[self.spec.tensor].to(torch.float32).contiguous()
+
+    def scale_output(self, vec):
+        """Multiplies what the norm gives by a vector, element by element (once, in the weight)."""
+        self.weight = self.weight * vec
 
     def add_forward(self, h, delta, out, rows=None):
         """h (float32 residual stream) += delta (a tensor, a ``csrc.api.Partial`` or None; a ``NormedDelta`` goes
@@ -111,26 +130,42 @@ register_part(GroupRMSNormSpec, GroupRMSNorm)
 
 
 class LayerNorm(Part):
-    """Layer norm with a weight and no bias, y = w * (x - mean) / sqrt(variance + eps), the variance the mean of the squared
-    deviations (taken of the deviations themselves, not of the squares). Statistics in float32, weight held in float32. It
+    """Layer norm with a weight and, where the spec names one, a bias: y = w * (x - mean) / sqrt(variance + eps) + b, the
+    variance the mean of the squared deviations (taken of the deviations themselves, not of the squares). Statistics in
+    float32, weight and bias held in float32. It
     runs in the kernel that adds a sublayer's output to the stream: as the norm of that output (``OutputNormBlock``) and as
     the norm behind the sum (``add_forward``)."""
     takes_partial = True
     takes_normed = True      # add_forward also takes a sublayer's output that has a norm of its own (NormedDelta)
+    takes_reset = True       # ... and a stream that starts anew (StreamReset)
+    bias = None
 
     def param_decls(self):
-        return [ParamDecl(self.spec.tensor, (self.spec.dim,), init="norm", keep_float32=True)]
+        d = [ParamDecl(self.spec.tensor, (self.spec.dim,), init="norm", keep_float32=True)]
+        if self.spec.bias is not None:
+            d.append(ParamDecl(self.spec.bias, (self.spec.dim,), init="around_zero", keep_float32=True))
+        return d
 
     def bind(self, tensors):
         self.weight = tensors[self.spec.tensor].to(torch.float32).contiguous()
+        if self.spec.bias is not None:
+            self.bias = tensors[self.spec.bias].to(torch.float32).contiguous()
+
+    def scale_output(self, vec):
+        self.weight = self.weight * vec
+        if self.bias is not None:
+            self.bias = self.bias * vec
 
     def args(self):
-        """(weight, eps, center) as ``csrc.api.sublayer_add`` takes a norm."""
-        return self.weight, self.spec.eps, True
+        """(weight, eps, center, bias) as ``csrc.api.sublayer_add`` takes a norm."""
+        return self.weight, self.spec.eps, True, self.bias
 
     def add_forward(self, h, delta, out, rows=None):
         """h += delta, out = norm(h); with ``rows`` of those rows only, leaving h as it is."""
         norm = None
+        if isinstance(delta, StreamReset):
+            api.sublayer_add(None, delta.delta, None, out, h_out=h, next_norm=self.args(), base=delta.base)
+            return out
         if isinstance(delta, NormedDelta):
             delta, norm = delta.delta, norm_args(delta.norm)
         api.sublayer_add(h, delta, norm, out, h_out=h if rows is None else None, rows=rows, next_norm=self.args())
@@ -141,7 +176,7 @@ register_part(LayerNormSpec, LayerNorm)
 
 
 def norm_args(norm):
-    """(weight, eps, center) of a norm part, as ``csrc.api.sublayer_add`` takes it."""
+    """A norm part as ``csrc.api.sublayer_add`` takes it: (weight, eps, center), or with the bias behind them."""
     if isinstance(norm, LayerNorm):
         return norm.args()
     if isinstance(norm, RMSNorm):

@@ -5,6 +5,7 @@ Adding an architecture: write a ``ModelConfig`` subclass with ``architecture``, 
 ``to_dict`` and ``to_spec``, then ``register_architecture(YourConfig)``."""
 from .config.base import ConfigError, read_config_json
 from .config.fukatar import FukatarConfig
+from .config.mozutar import MozutarConfig
 from .config.nevotar import NevotarConfig
 from .config.nilivik import NilivikConfig
 from .config.pibulix import PibulixConfig
@@ -51,3 +52,4 @@ register_architecture(PibulixConfig)
 register_architecture(VenidraConfig)
 register_architecture(NevotarConfig)
 register_architecture(FukatarConfig)
+register_architecture(MozutarConfig)
