@@ -1134,8 +1134,173 @@ def fukatar_kernel_times(torch, dk, pk, cfg_d, p_cfg):
     return out
 
 
+def mozutar_config(width, heads, kv_heads, ff_qwen, layers, vocab):
+    """A Mozutar model of Qwen3's width with ``layers`` layer runs: first and last a matrix-memory layer (half Qwen3's heads, of
+    128 x 128) with a dense feed-forward of Qwen3's size; between them half as many layers as there are runs left, run twice:
+    attention of Qwen3's head counts (heads of 128 rotated whole, capped scores, keys as values) beside gated linear attention
+    (half as many heads of 128 x 128), with a mixture of 30 experts and 2 identity experts in 4 groups, of which a token uses 4
+    from 2 groups, each expert a quarter of Qwen3's feed-forward."""
+    hd, gh = 128, heads // 2
+    eff = max(64, ff_qwen // 4 // 64 * 64)
+    mem = {"type": "mlstm", "mixer": {"heads": gh, "dim": hd, "vdim": hd, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": ff_qwen}}
+    par = {"type": "parallel",
+           "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 50.0, "rot": {"dims": hd, "base": 1e6}},
+                     "right": {"heads": gh, "dim": hd, "vdim": hd, "tau": 16.0}},
+           "mlp": {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": 30, "identity": 2, "top": 4, "groups": {"count": 4, "keep": 2}}}}
+    inner = max(1, (layers - 2) // 2)
+    return dict(architecture="Mozutar", vocab=vocab, width=width, norm={"eps": 1e-6}, embedding={"scale": width ** 0.5},
+                loop={"start": 1, "stop": 1 + inner, "times": 2}, layers=[mem] + [par] * inner + [mem])
+
+
+def mozutar_kernel_times(torch, dk, pk, cfg_d, p_cfg):
+    """The design's steps alone (the parts of a model of ``cfg_d``, so each step runs whichever kernel the part picks), beside
+    the like steps of the Pibulix model ``p_cfg`` of the same width: CUDA events around one step, L2 flushed before each (a 256
+    MB write), median of 5 after 2 untimed. Prompts' attention, experts and products against the bfloat16 peak, everything else
+    against the copy peak by the bytes the step must move."""
+    from dryft_challenge_htn_2026_b200.cache import Cache
+    from dryft_challenge_htn_2026_b200.csrc import api
+    from dryft_challenge_htn_2026_b200.engine.batch import build_context
+    from dryft_challenge_htn_2026_b200.parts import Runtime, build_part
+    from dryft_challenge_htn_2026_b200.parts.linear import linear, linear_partial
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
+
+    def timed(fn):
+        ts = []
+        for i in range(7):
+            flush.fill_(float(i))
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        return statistics.median(ts[2:]) * 1e3        # microseconds
+
+    def flops_rec(us, flops):
+        return {"us": round(us, 1), "tflops": round(flops / us / 1e6, 1), "frac_bf16": round(flops / us / 1e6 / pk["bf16_tflops"], 4)}
+
+    def bytes_rec(us, moved):
+        return {"us": round(us, 1), "gbs": round(moved / us / 1e3, 1), "frac_hbm": round(moved / us / 1e3 / pk["hbm_gbs"], 4)}
+
+    rt = Runtime(dev, bf)
+    g = torch.Generator(device=dev).manual_seed(1)
+    spec, pspec = dk.config_from_dict(cfg_d).to_spec(), dk.config_from_dict(p_cfg).to_spec()
+    W = spec.hidden_size
+
+    def bound(part_spec):
+        part = build_part(part_spec, rt)
+        part.bind({d.name: (torch.randn(d.shape, generator=g, device=dev) * (0.2 if d.init in ("wide", "taps") else 0.02) + (1.0 if d.init == "norm" else 0.0)).to(
+            torch.float32 if d.keep_float32 else bf) for d in part.param_decls()})
+        part.prepare(16384)
+        return part
+
+    mem, par = bound(spec.layers[0].mixer), bound(spec.layers[1].mixer)
+    att, gla = par.branches[0][1], par.branches[1][1]
+    p_att, p_gla = bound(pspec.layers[0].mixer), bound(pspec.layers[1].mixer)
+    moe, p_moe = bound(spec.layers[1].feed_forward), bound(pspec.layers[1].feed_forward)
+    p_norm = bound(pspec.layers[0].norm_mix)
+    window, ms = p_att.spec.window, mem.spec
+    w, b = torch.ones(W, device=dev), torch.zeros(W, device=dev)
+    w_take = (torch.randn(W, 2 * W, generator=g, device=dev) * 0.02).to(bf)
+    out, scratch = {}, {}
+
+    class Ctx:
+        def scratch(self, key, make):
+            if key not in scratch:
+                scratch[key] = make()
+            return scratch[key]
+
+    def fill(cache, n):
+        for e in range(n):
+            for v in cache.views(e):
+                if hasattr(v, "k"):
+                    v.k.normal_(), v.v.normal_()
+
+    def steps(ctx, cache, rows, tag, pairs, keys, p_pairs, p_keys):
+        """``pairs``: (query, key) pairs in sight in a prompt (0: single tokens that read ``keys`` keys each); ``p_*``: Pibulix's."""
+        ctx.carry = {}
+        rand = lambda n: (torch.randn(rows, n, device=dev) * 0.5).to(bf)
+        empty = lambda n: torch.empty(rows, n, dtype=bf, device=dev)
+        # the recurrences, from projection rows to gated rows: what a prompt must move (q, k, v, gate in, rows out), what a single token must (the state, twice)
+        proj, mid = rand(mem.n_in), empty(mem.n_mid)
+        us = timed(lambda: mem.mix(ctx, cache.views(0), proj, mid, 1.0))
+        out[f"matrix_memory_{tag}"] = bytes_rec(us, rows * ms.num_heads * (2 * ms.head_dim + 3 * ms.v_head_dim) * 2 if pairs else
+                                                rows * ms.num_heads * ms.head_dim * ms.v_head_dim * 4 * 2)
+        for name, part, views in (("gated_linear_attention", gla, cache.views(1)[1:]), ("pibulix_gated_linear_attention", p_gla, cache.views(3))):
+            gs, pg, mg = part.spec, rand(part.n_in), empty(part.n_mid)
+            us = timed(lambda: part.mix(ctx, views, pg, mg, 1.0))
+            out[f"{name}_{tag}"] = bytes_rec(us, rows * gs.num_heads * (2 * gs.head_dim + 3 * gs.v_head_dim) * 2 if pairs else
+                                             rows * gs.num_heads * gs.head_dim * gs.v_head_dim * 4 * 2)
+        # attention: rows between projection and cache, then the attention itself
+        s, proj, mid = att.spec, rand(att.n_in), empty(att.n_mid)
+        q = att.rotated_queries(ctx, cache.views(1)[:1], proj)
+        us = timed(lambda: att.rotated_queries(ctx, cache.views(1)[:1], proj))
+        out[f"rows_norm_rotation_cache_{tag}"] = bytes_rec(us, rows * (2 * att.n_q + 3 * att.n_k) * 2)
+        us = timed(lambda: att.attend(ctx, cache.views(1)[0], q, None, None, None, mid, 1.0, writes=False))
+        out[f"attention_{tag}"] = flops_rec(us, 4 * s.num_heads * s.head_dim * pairs) if pairs else \
+            dict(bytes_rec(us, rows * s.num_kv_heads * keys * 2 * s.head_dim * 2), keys=keys)
+        s, proj, mid = p_att.spec, rand(p_att.n_in), empty(p_att.n_mid)
+        x = p_att.prepared_rows(ctx, cache.views(2), proj)
+        us = timed(lambda: p_att.prepared_rows(ctx, cache.views(2), proj))
+        out[f"pibulix_rows_conv_norm_rotation_cache_{tag}"] = bytes_rec(us, rows * (2 * p_att.n_qkv + p_att.n_k + p_att.n_v) * 2)
+        us = timed(lambda: p_att.attend(ctx, cache.views(2)[0], x[:, :p_att.n_q], None, None, None, mid, 1.0, writes=False))
+        out[f"pibulix_attention_{tag}"] = flops_rec(us, 4 * s.num_heads * s.head_dim * p_pairs) if pairs else \
+            dict(bytes_rec(us, rows * s.num_kv_heads * p_keys * 2 * s.head_dim * 2), keys=p_keys)
+        # experts (identity experts do no arithmetic: of 32 outputs 30 are experts)
+        a = rand(W)
+        for name, part, share in (("experts", moe, 30 / 32), ("pibulix_experts", p_moe, 1.0)):
+            e = part.spec
+            shared = 1 if e.shared_ff else 0
+            us = timed(lambda: part.forward(Ctx(), a))
+            read = (min(e.num_experts, rows * e.top * share) + shared) * 3 * e.expert_ff * W * 2
+            out[f"{name}_{tag}"] = flops_rec(us, rows * (e.top * share + shared) * 6 * e.expert_ff * W) if pairs else bytes_rec(us, read)
+        # the stream
+        h, o, d2 = torch.randn(rows, W, device=dev), empty(W), rand(W)
+        norm = (w, 1e-6, True, b)
+        us = timed(lambda: api.sublayer_add(h, a, norm, o, h_out=h, next_norm=norm))
+        out[f"output_norm_sum_norm_{tag}"] = bytes_rec(us, rows * W * (4 + 2 + 4 + 2))
+        two = api.NormedSum([a, d2], [w, w], 1e-6, 0.5)
+        us = timed(lambda: api.sublayer_add(h, two, norm, o, h_out=h, next_norm=norm))
+        out[f"two_output_norms_sum_norm_{tag}"] = bytes_rec(us, rows * W * (4 + 4 + 4 + 2))
+        us = timed(lambda: p_norm.scale_add_forward(h, 1.0, a, o))
+        out[f"pibulix_norm_{tag}"] = bytes_rec(us, rows * W * (4 + 4 + 2 + 2))
+        both = rand(2 * W)
+        us = timed(lambda: linear_partial(both, w_take))
+        out[f"embedding_taken_in_{tag}"] = flops_rec(us, 2 * rows * 2 * W * W) if pairs else bytes_rec(us, 2 * W * W * 2)
+        us = timed(lambda: linear(both, w_take))
+        out[f"plain_product_of_the_same_size_{tag}"] = flops_rec(us, 2 * rows * 2 * W * W) if pairs else bytes_rec(us, 2 * W * W * 2)
+        new = linear_partial(both, w_take)
+        us = timed(lambda: api.sublayer_add(None, new, None, o, h_out=h, next_norm=norm, base=b))
+        out[f"stream_anew_norm_{tag}"] = bytes_rec(us, rows * W * (4 * new.ws.shape[0] + 4 + 2))
+
+    entries = [mem.cache_requests(), par.cache_requests(), p_att.cache_requests(), p_gla.cache_requests()]
+    plans = list({p.key: p for part in (mem, par, p_att) for p in part.step_plans()}.values())
+    for tokens in (2048, 8192):
+        cache = Cache(entries, tokens + 64, 2, dev)
+        slot = cache.begin()
+        ctx = build_context(cache, [(slot, [0] * tokens, [])], dev, plans=plans)
+        fill(cache, 4)
+        steps(ctx, cache, tokens, str(tokens), tokens * (tokens + 1) // 2, 0, sum(min(i + 1, window) for i in range(tokens)), 0)
+        cache.end(slot)
+        del cache
+    for batch in (8, 64):
+        context = 3000
+        cache = Cache(entries, batch * (context + 64), batch, dev)
+        slots = [cache.begin() for _ in range(batch)]
+        for sl in slots:
+            cache.reserve(sl, context + 1)
+            cache.length[sl] = context
+        ctx = build_context(cache, [(sl, [0], []) for sl in slots], dev, plans=plans)
+        fill(cache, 4)
+        steps(ctx, cache, batch, f"decode_b{batch}", 0, context + 1, 0, min(window, context + 1) + p_att.spec.keep_first)
+        del cache
+    torch.cuda.empty_cache()
+    return out
+
+
 def run_design(args):
-    """``--design nilivik`` / ``--design pibulix`` / ``--design venidra`` / ``--design nevotar`` / ``--design fukatar``: prefill and decode of that decoder at Qwen3 layer sizes (random weights,
+    """``--design nilivik`` / ``--design pibulix`` / ``--design venidra`` / ``--design nevotar`` / ``--design fukatar`` / ``--design mozutar``: prefill and decode of that decoder at Qwen3 layer sizes (random weights,
     ``--layers`` layers, default 4) beside Qwen3 itself at the same width, layer count and parameters a
     layer, and the design's mixer kernels alone beside Qwen3's attention kernels. One JSON line."""
     import torch
@@ -1148,13 +1313,19 @@ def run_design(args):
     layers = args.layers or 4
     chunk = 2048
     vocab = 32768
-    out = {"design": args.design, "beside": {"nevotar": "Pibulix", "fukatar": "Venidra"}.get(args.design, "Qwen3ForCausalLM"), "layers": layers, "chunk": chunk, "vocab": vocab, "dtype": "bf16",
+    out = {"design": args.design, "beside": {"nevotar": "Pibulix", "fukatar": "Venidra", "mozutar": "Pibulix"}.get(args.design, "Qwen3ForCausalLM"), "layers": layers, "chunk": chunk, "vocab": vocab, "dtype": "bf16",
            "data": "synthetic: random weights, uniform random token ids", "peaks": pk, "sizes": {}}
     for size in args.design_sizes.split(","):
         q = dict(SIZES[size]["config"], num_hidden_layers=layers, vocab_size=vocab, tie_word_embeddings=True)
         beside = ("qwen3", q)
         sizes = (q["hidden_size"], q["num_attention_heads"], q["num_key_value_heads"], q["intermediate_size"], layers, vocab)
-        if args.design == "fukatar":
+        if args.design == "mozutar":
+            n = mozutar_config(*sizes)
+            beside = ("pibulix", pibulix_config(*sizes, PIBULIX_WINDOW))
+            rec = {"width": q["hidden_size"], "expert_ff": n["layers"][1]["mlp"]["expert"]["ff"], "window": PIBULIX_WINDOW,
+                   "beside": "Pibulix of the same width, layer runs and feed-forward arithmetic (the closest of the library's designs: "
+                             "gated linear attention, capped attention, a mixture of experts)"}
+        elif args.design == "fukatar":
             n = fukatar_config(*sizes)
             beside = ("venidra", venidra_config(*sizes))
             rec = {"width": q["hidden_size"], "ff": n["layers"][0]["mlp"]["ff"], "kv_rank": 512,
@@ -1192,7 +1363,9 @@ def run_design(args):
             rec[name] = r
             del model
             torch.cuda.empty_cache()
-        if args.design == "fukatar":
+        if args.design == "mozutar":
+            rec["kernels"] = mozutar_kernel_times(torch, dk, pk, n, beside[1])
+        elif args.design == "fukatar":
             rec["kernels"] = fukatar_kernel_times(torch, dk, pk, n, pibulix_config(*sizes, PIBULIX_WINDOW))
             rec["venidra_kernels"] = venidra_kernel_times(torch, dk, pk, beside[1], q["num_attention_heads"], q["num_key_value_heads"])
         elif args.design == "nevotar":
@@ -1410,9 +1583,9 @@ def main():
     ap.add_argument("--prefill-only", action="store_true", help="only the 2,048-token prefill (for profiling its kernels)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="with --prefill-only: a prompt of another length")
     ap.add_argument("--pdl", type=int, default=1, help="programmatic dependent launch on (1) or off (0)")
-    ap.add_argument("--design", default=None, choices=["nilivik", "pibulix", "venidra", "nevotar", "fukatar"],
+    ap.add_argument("--design", default=None, choices=["nilivik", "pibulix", "venidra", "nevotar", "fukatar", "mozutar"],
                     help="instead of the default workload: prefill and decode of this design at Qwen3 layer sizes beside Qwen3 "
-                         "itself at equal size (nevotar: beside Pibulix, fukatar: beside Venidra, the closest of the library's designs), and its mixer "
+                         "itself at equal size (nevotar and mozutar: beside Pibulix, fukatar: beside Venidra, the closest of the library's designs), and its mixer "
                          "kernels alone (one JSON line of its own)")
     ap.add_argument("--design-sizes", default="4b,8b", help="with --design: which of the layer sizes")
     args = ap.parse_args()

@@ -1850,15 +1850,30 @@ def _need_memory(q, k, v, i_rows, f_rows, i_bias, f_bias, states, n_heads, head_
         raise KernelError(f"{what}: shapes do not match (columns of one matrix, key sizes up to 256)")
 
 
+MEMORY_CHUNK = 256               # tokens a chunk of the tensor-core form of a matrix memory
+
+
+def memory_chunks_take(head_dim, v_head_dim):
+    """Head sizes of the tensor-core form: keys and values in steps of 16 up to 128."""
+    return all(d % 16 == 0 and 16 <= d <= 128 for d in (head_dim, v_head_dim))
+
+
+def memory_chunk_operands(q, k, v, gate, out):
+    return q.dtype == torch.bfloat16 and q.stride(0) % 8 == 0 and out.stride(0) % 2 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, k, v)) \
+        and gate.data_ptr() % 4 == 0 and out.data_ptr() % 4 == 0
+
+
 def matrix_memory(q, k, v, gate, i_rows, f_rows, i_bias, f_bias, cap, states, weight, eps, out_scale, out, q_scale, cu_q, seq_pos0, seq_slot,
-                  row_pos, n_seq, n_heads, head_dim, v_head_dim):
+                  row_pos, n_seq, n_heads, head_dim, v_head_dim, chunks=None):
     """The matrix memory with exponential gates over a step's rows, all float32 behind the projection: log gates i = cap
     tanh((i_rows + i_bias) / cap), f = log sigmoid of the same form; m' = max(f + m, i); S <- exp(f + m - m') S + exp(i - m')
     k v^T, n likewise with k alone; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6) with q times ``q_scale``; ``out`` = each head's
     o over its root mean square (``eps`` inside the root) * ``weight`` [heads * v_head_dim] * sigmoid(gate) * ``out_scale``.
     ``states`` = (S [slots, heads, D, V], n [slots, heads, D], m [slots, heads]), float32, moved on. Rows of sequence s are
     cu_q[s] .. cu_q[s + 1]; ``cu_q`` None: row s alone, seq_pos0[s] < 0 marks padding. Single tokens are one kernel, portions
-    three (gates, recurrence, output)."""
+    three (gates, recurrence, output), or four on the tensor cores (gates, then chunks of ``MEMORY_CHUNK`` tokens side by side)
+    where ``chunks`` is given: int32 [n_seq + n_chunks, 4] = per sequence (its first chunk, how many), per chunk (sequence, first
+    row, rows, number within the sequence); head sizes as ``memory_chunks_take`` says and rows on 16-byte boundaries."""
     _need_memory(q, k, v, i_rows, f_rows, i_bias, f_bias, states, n_heads, head_dim, v_head_dim, "matrix_memory")
     _need_rows(gate, "gate", q.dtype), _need_rows(out, "out", q.dtype), _need(weight, "weight", torch.float32, 1)
     for t, nm in ((cu_q, "cu_q"), (seq_pos0, "seq_pos0"), (seq_slot, "seq_slot"), (row_pos, "row_pos")):
@@ -1874,9 +1889,21 @@ def matrix_memory(q, k, v, gate, i_rows, f_rows, i_bias, f_bias, cap, states, we
                                           _p(S), _p(n), _p(m), _p(weight), c_float(eps), c_float(out_scale), _p(out), c_longlong(out.stride(0)),
                                           _p(seq_pos0), _p(seq_slot), c_float(q_scale), T, *sizes, _stream()), "matrix_memory")
     scal = torch.empty((T, n_heads, 4), dtype=torch.float32, device=q.device)
-    o = torch.empty((T, n_mid), dtype=torch.float32, device=q.device)
+    tiled = chunks is not None and memory_chunks_take(head_dim, v_head_dim) and memory_chunk_operands(q, k, v, gate, out)
     _check(lib, lib.dk_mm_gates(_dt(q), _p(i_rows), _p(f_rows), ld, _p(i_bias), _p(f_bias), c_float(cap), _p(scal), _p(m), _p(cu_q), _p(seq_pos0),
-                                _p(seq_slot), n_seq, n_heads, _stream()), "matrix_memory gates")
+                                _p(seq_slot), n_seq, n_heads, MEMORY_CHUNK if tiled else 0, _stream()), "matrix_memory gates")
+    if tiled:
+        _need(chunks, "chunks", torch.int32, 2)
+        nc = chunks.shape[0] - n_seq
+        if nc < 1 or chunks.shape[1] != 4:
+            raise KernelError("matrix_memory: a list of chunks without chunks")
+        u = torch.empty((nc, n_heads, head_dim, v_head_dim + 8), dtype=torch.float32, device=q.device)
+        planes = torch.empty((nc, n_heads, 2, head_dim, v_head_dim + 8), dtype=torch.bfloat16, device=q.device)
+        lib = _lib("matrix_memory_bf16.cu", {"HD": head_dim, "HDV": v_head_dim})
+        return _check(lib, lib.dk_mm_chunks(_p(q), _p(k), _p(v), _p(gate), ld, _p(scal), _p(chunks), n_seq, nc, _p(u), _p(planes), _p(S), _p(n),
+                                            _p(seq_slot), _p(weight), c_float(eps), c_float(q_scale), c_float(out_scale), _p(out),
+                                            c_longlong(out.stride(0)), n_heads, _stream()), "matrix_memory chunks", 3)
+    o = torch.empty((T, n_mid), dtype=torch.float32, device=q.device)
     _check(lib, lib.dk_mm_portion(_dt(q), _p(q), _p(k), _p(v), ld, _p(scal), _p(o), _p(S), _p(n), _p(cu_q), _p(seq_pos0), _p(seq_slot),
                                   c_float(q_scale), n_seq, *sizes, _stream()), "matrix_memory")
     _check(lib, lib.dk_mm_output(_dt(q), _p(o), _p(scal), _p(weight), c_float(eps), _p(gate), ld, c_float(out_scale), _p(out),

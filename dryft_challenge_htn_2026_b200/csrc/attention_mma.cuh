@@ -47,6 +47,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// A fragment (16 rows m0.., 16 columns k0..) of the transpose of a matrix stored [k][m] with row stride KSTR:
+// the four 8x8 blocks (m0,k0), (m0+8,k0), (m0,k0+8), (m0+8,k0+8) come from the stored blocks with rows and
+// columns exchanged, each loaded transposed.
+__device__ __forceinline__ void ldsm_a_transposed(uint32_t (&a)[4], const bf16* base, int k0, int m0) {
+    const int lane = threadIdx.x & 31, i = lane & 7, blk = lane >> 3;
+    ldsm_x4_trans(a, base + (k0 + i + 8 * (blk >> 1)) * KSTR + m0 + 8 * (blk & 1));
+}
+
 // Q fragments of 16 rows; row_ptr0/1: the rows of lane group g and g+8 (nullptr: row of zeros).
 __device__ __forceinline__ void load_q_frags(uint32_t (&qf)[HD / 16][4], const bf16* row0, const bf16* row1) {
     const int t = threadIdx.x & 3;

@@ -70,14 +70,6 @@ __device__ __forceinline__ void stage_weighted_keys(bf16* hi, bf16* lo, const bf
     }
 }
 
-// A fragment (16 rows m0.., 16 columns k0..) of the transpose of a matrix stored [k][m] with row stride KSTR:
-// the four 8x8 blocks (m0,k0), (m0+8,k0), (m0,k0+8), (m0+8,k0+8) come from the stored blocks with rows and
-// columns exchanged, each loaded transposed.
-__device__ __forceinline__ void ldsm_a_transposed(uint32_t (&a)[4], const bf16* base, int k0, int m0) {
-    const int lane = threadIdx.x & 31, i = lane & 7, blk = lane >> 3;
-    ldsm_x4_trans(a, base + (k0 + i + 8 * (blk >> 1)) * KSTR + m0 + 8 * (blk & 1));
-}
-
 constexpr int LC_THREADS = 256;   // warps 0-3: the block's outputs, 16 rows each; warps 4-7: the state and its update
 
 template <int DVB>

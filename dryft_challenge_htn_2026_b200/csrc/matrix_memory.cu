@@ -7,6 +7,7 @@
 // q, k, v, gate and the two gate rows are columns of one projection in the storage type; everything else is float32.
 //
 // Portions run in three kernels:
+// (bfloat16 portions of suitable sizes go on to matrix_memory_bf16.cu behind the first of them):
 //   * mm_gates: a warp per (sequence, head). A token maps m to max(f + m, i); two such maps in a row are another one,
 //     (f1 + f2, max(i1 + f2, i2)), so 32 tokens' running maxima come from five shuffles. Leaves per (token, head) what the
 //     recurrence multiplies by: exp(f + m - m'), exp(i - m'), exp(-m').
@@ -24,11 +25,12 @@ __device__ __forceinline__ float mm_cap(float x, float cap) { return cap * tanhf
 __device__ __forceinline__ float mm_log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
 // ------------------------------------------------------------------------------------------------ gates of a portion
-// scal [tokens, heads, 4] = (exp(f + m - m'), exp(i - m'), exp(-m'), -); the last number is n . q, from mm_portion
+// scal [tokens, heads, 4] = (exp(f + m - m'), exp(i - m'), exp(-m'), -); the last number is n . q, from mm_portion. With
+// ``chunk`` (a multiple of 32) the first number is the sum of (f + m - m') log2(e) from the first token of the token's chunk on.
 template <typename T>
 __global__ void __launch_bounds__(128)
 mm_gates_kernel(const T* irow, const T* frow, long long ld, const float* __restrict__ ibias, const float* __restrict__ fbias, float cap,
-                float4* scal, float* m_state, const int* cu_q, const int* seq_pos0, const int* seq_slot, int n_seq, int nh) {
+                float4* scal, float* m_state, const int* cu_q, const int* seq_pos0, const int* seq_slot, int n_seq, int nh, int chunk) {
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, item = blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -39,7 +41,7 @@ mm_gates_kernel(const T* irow, const T* frow, long long ld, const float* __restr
     float* mp = m_state + (size_t)seq_slot[s] * nh + h;
     float m = *mp;
     const float ib = ibias[h], fb = fbias[h];
-    float iz = 0.f, fz = 0.f;
+    float iz = 0.f, fz = 0.f, so_far = 0.f;
     auto fetch = [&](int t) {
         iz = t < r1 ? to_f(irow[(size_t)t * ld + h]) : 0.f;
         fz = t < r1 ? to_f(frow[(size_t)t * ld + h]) : 0.f;
@@ -63,7 +65,21 @@ mm_gates_kernel(const T* irow, const T* frow, long long ld, const float* __restr
         const float mt = fmaxf(F + m, I);
         float before = __shfl_up_sync(0xffffffffu, mt, 1);
         if (lane == 0) before = m;
-        if (on) scal[(size_t)(t0 + lane) * nh + h] = make_float4(expf(f + before - mt), expf(i - mt), expf(-mt), 0.f);
+        float keep = f + before - mt;
+        if (chunk) {
+            if ((t0 - r0) % chunk == 0) so_far = 0.f;
+            keep *= 1.4426950408889634f;
+#pragma unroll
+            for (int d = 1; d < 32; d <<= 1) {
+                const float x = __shfl_up_sync(0xffffffffu, keep, d);
+                if (lane >= d) keep += x;
+            }
+            keep += so_far;
+            so_far = __shfl_sync(0xffffffffu, keep, 31);
+        } else {
+            keep = expf(keep);
+        }
+        if (on) scal[(size_t)(t0 + lane) * nh + h] = make_float4(keep, expf(i - mt), expf(-mt), 0.f);
         m = __shfl_sync(0xffffffffu, mt, 31);
     }
     if (lane == 0) *mp = m;
@@ -406,13 +422,14 @@ mm_step_kernel(const T* q, const T* k, const T* v, const T* gate, const T* irow,
 
 DK_EXPORT int dk_mm_gates(int dtype, const void* irow, const void* frow, long long ld, const float* ibias, const float* fbias, float cap,
                           void* scal, float* m_state, const int* cu_q, const int* seq_pos0, const int* seq_slot, int n_seq, int nh,
-                          cudaStream_t st) {
+                          int chunk, cudaStream_t st) {
+    if (chunk < 0 || chunk % 32) return (int)cudaErrorInvalidValue;
     const dim3 grid((n_seq * nh + 3) / 4), block(128);
     if (dtype == 0)
         return dk_launch(mm_gates_kernel<float>, grid, block, 0, st, (const float*)irow, (const float*)frow, ld, ibias, fbias, cap, (float4*)scal,
-                         m_state, cu_q, seq_pos0, seq_slot, n_seq, nh);
+                         m_state, cu_q, seq_pos0, seq_slot, n_seq, nh, chunk);
     return dk_launch(mm_gates_kernel<bf16>, grid, block, 0, st, (const bf16*)irow, (const bf16*)frow, ld, ibias, fbias, cap, (float4*)scal, m_state,
-                     cu_q, seq_pos0, seq_slot, n_seq, nh);
+                     cu_q, seq_pos0, seq_slot, n_seq, nh, chunk);
 }
 
 template <typename T>
