@@ -1891,7 +1891,7 @@ def matrix_memory(q, k, v, gate, i_rows, f_rows, i_bias, f_bias, cap, states, we
     scal = torch.empty((T, n_heads, 4), dtype=torch.float32, device=q.device)
     tiled = chunks is not None and memory_chunks_take(head_dim, v_head_dim) and memory_chunk_operands(q, k, v, gate, out)
     _check(lib, lib.dk_mm_gates(_dt(q), _p(i_rows), _p(f_rows), ld, _p(i_bias), _p(f_bias), c_float(cap), _p(scal), _p(m), _p(cu_q), _p(seq_pos0),
-                                _p(seq_slot), n_seq, n_heads, MEMORY_CHUNK if tiled else 0, _stream()), "matrix_memory gates")
+                                _p(seq_slot), n_seq, n_heads, MEMORY_CHUNK if tiled else 0, c_longlong(T), _stream()), "matrix_memory gates")
     if tiled:
         _need(chunks, "chunks", torch.int32, 2)
         nc = chunks.shape[0] - n_seq

@@ -8,8 +8,9 @@
 //
 // Portions run in three kernels:
 // (bfloat16 portions of suitable sizes go on to matrix_memory_bf16.cu behind the first of them):
-//   * mm_gates: a warp per (sequence, head). A token maps m to max(f + m, i); two such maps in a row are another one,
-//     (f1 + f2, max(i1 + f2, i2)), so 32 tokens' running maxima come from five shuffles. Leaves per (token, head) what the
+//   * mm_gates: a block per (sequence, head). A token maps m to max(f + m, i); two such maps in a row are another one,
+//     (f1 + f2, max(i1 + f2, i2)), so a warp's 32 running maxima come from five shuffles, and a block's from five more over its
+//     warps' maps. Leaves per (token, head) what the
 //     recurrence multiplies by: exp(f + m - m'), exp(i - m'), exp(-m').
 //   * mm_portion: the recurrence over the portion, columns of S in registers, rows staged ahead by cp.async.
 //   * mm_output: quotient, norm, weight, gate; a warp per (token, head).
@@ -26,63 +27,85 @@ __device__ __forceinline__ float mm_log_sigmoid(float x) { return fminf(x, 0.f) 
 
 // ------------------------------------------------------------------------------------------------ gates of a portion
 // scal [tokens, heads, 4] = (exp(f + m - m'), exp(i - m'), exp(-m'), -); the last number is n . q, from mm_portion. With
-// ``chunk`` (a multiple of 32) the first number is the sum of (f + m - m') log2(e) from the first token of the token's chunk on.
+// ``chunk`` (a multiple of 32, the block's threads a multiple of it) the first number is the sum of (f + m - m') log2(e) from the
+// first token of the token's chunk on.
+struct MaxMap {          // m -> max(f + m, i)
+    float f, i;
+};
+// the maps of the lanes up to this one, in order
+__device__ __forceinline__ MaxMap warp_maps(MaxMap a, int lane) {
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+        const float f1 = __shfl_up_sync(0xffffffffu, a.f, d), i1 = __shfl_up_sync(0xffffffffu, a.i, d);
+        if (lane >= d) {
+            a.i = fmaxf(i1 + a.f, a.i);
+            a.f += f1;
+        }
+    }
+    return a;
+}
+
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(1024)
 mm_gates_kernel(const T* irow, const T* frow, long long ld, const float* __restrict__ ibias, const float* __restrict__ fbias, float cap,
-                float4* scal, float* m_state, const int* cu_q, const int* seq_pos0, const int* seq_slot, int n_seq, int nh, int chunk) {
+                float4* scal, float* m_state, const int* cu_q, const int* seq_pos0, const int* seq_slot, int nh, int chunk) {
+    __shared__ MaxMap maps[32];
+    __shared__ float sums[32], m_next;
     pdl_wait();
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, item = blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (item >= n_seq * nh) return;
-    const int s = item / nh, h = item % nh;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
+    const int s = blockIdx.x, h = blockIdx.y;
     if (seq_pos0[s] < 0) return;
     const int r0 = cu_q[s], r1 = cu_q[s + 1];
     float* mp = m_state + (size_t)seq_slot[s] * nh + h;
     float m = *mp;
     const float ib = ibias[h], fb = fbias[h];
-    float iz = 0.f, fz = 0.f, so_far = 0.f;
+    float iz = 0.f, fz = 0.f;
     auto fetch = [&](int t) {
-        iz = t < r1 ? to_f(irow[(size_t)t * ld + h]) : 0.f;
-        fz = t < r1 ? to_f(frow[(size_t)t * ld + h]) : 0.f;
+        if (t < r1) {
+            iz = to_f(irow[(size_t)t * ld + h]);
+            fz = to_f(frow[(size_t)t * ld + h]);
+        }
     };
-    fetch(r0 + lane);
-    for (int t0 = r0; t0 < r1; t0 += 32) {
-        const bool on = t0 + lane < r1;
+    fetch(r0 + tid);
+    for (int t0 = r0; t0 < r1; t0 += blockDim.x) {
+        const bool on = t0 + tid < r1;
         // past the end: the map that leaves m alone
         const float i = on ? mm_cap(iz + ib, cap) : -INFINITY;
         const float f = on ? mm_log_sigmoid(mm_cap(fz + fb, cap)) : 0.f;
-        fetch(t0 + 32 + lane);
-        float F = f, I = i;
-#pragma unroll
-        for (int d = 1; d < 32; d <<= 1) {
-            const float F1 = __shfl_up_sync(0xffffffffu, F, d), I1 = __shfl_up_sync(0xffffffffu, I, d);
-            if (lane >= d) {
-                I = fmaxf(I1 + F, I);
-                F += F1;
-            }
+        fetch(t0 + blockDim.x + tid);
+        const MaxMap a = warp_maps({f, i}, lane);
+        if (lane == 31) maps[warp] = a;
+        __syncthreads();
+        if (warp == 0) {
+            const MaxMap all = warp_maps(lane < n_warps ? maps[lane] : MaxMap{0.f, -INFINITY}, lane);
+            maps[lane] = all;
         }
-        const float mt = fmaxf(F + m, I);
+        __syncthreads();
+        const float ahead = warp == 0 ? m : fmaxf(maps[warp - 1].f + m, maps[warp - 1].i);        // the maximum ahead of this warp
+        const float mt = fmaxf(a.f + ahead, a.i);
         float before = __shfl_up_sync(0xffffffffu, mt, 1);
-        if (lane == 0) before = m;
+        if (lane == 0) before = ahead;
         float keep = f + before - mt;
         if (chunk) {
-            if ((t0 - r0) % chunk == 0) so_far = 0.f;
             keep *= 1.4426950408889634f;
 #pragma unroll
             for (int d = 1; d < 32; d <<= 1) {
                 const float x = __shfl_up_sync(0xffffffffu, keep, d);
                 if (lane >= d) keep += x;
             }
-            keep += so_far;
-            so_far = __shfl_sync(0xffffffffu, keep, 31);
+            if (lane == 31) sums[warp] = keep;
+            __syncthreads();
+            for (int w = warp / (chunk / 32) * (chunk / 32); w < warp; w++) keep += sums[w];
         } else {
             keep = expf(keep);
         }
-        if (on) scal[(size_t)(t0 + lane) * nh + h] = make_float4(keep, expf(i - mt), expf(-mt), 0.f);
-        m = __shfl_sync(0xffffffffu, mt, 31);
+        if (on) scal[(size_t)(t0 + tid) * nh + h] = make_float4(keep, expf(i - mt), expf(-mt), 0.f);
+        if (tid == (int)blockDim.x - 1) m_next = mt;
+        __syncthreads();              // also: maps and sums may be written again
+        m = m_next;
     }
-    if (lane == 0) *mp = m;
+    if (tid == 0) *mp = m;
 }
 
 // --------------------------------------------------------------------------------------------- recurrence of a portion
@@ -422,14 +445,14 @@ mm_step_kernel(const T* q, const T* k, const T* v, const T* gate, const T* irow,
 
 DK_EXPORT int dk_mm_gates(int dtype, const void* irow, const void* frow, long long ld, const float* ibias, const float* fbias, float cap,
                           void* scal, float* m_state, const int* cu_q, const int* seq_pos0, const int* seq_slot, int n_seq, int nh,
-                          int chunk, cudaStream_t st) {
-    if (chunk < 0 || chunk % 32) return (int)cudaErrorInvalidValue;
-    const dim3 grid((n_seq * nh + 3) / 4), block(128);
+                          int chunk, long long n_rows, cudaStream_t st) {
+    if (chunk < 0 || chunk % 32 || (chunk && 256 % chunk)) return (int)cudaErrorInvalidValue;
+    const dim3 grid(n_seq, nh), block(n_rows > 256LL * n_seq ? 1024 : 256);
     if (dtype == 0)
         return dk_launch(mm_gates_kernel<float>, grid, block, 0, st, (const float*)irow, (const float*)frow, ld, ibias, fbias, cap, (float4*)scal,
-                         m_state, cu_q, seq_pos0, seq_slot, n_seq, nh, chunk);
+                         m_state, cu_q, seq_pos0, seq_slot, nh, chunk);
     return dk_launch(mm_gates_kernel<bf16>, grid, block, 0, st, (const bf16*)irow, (const bf16*)frow, ld, ibias, fbias, cap, (float4*)scal, m_state,
-                     cu_q, seq_pos0, seq_slot, n_seq, nh, chunk);
+                     cu_q, seq_pos0, seq_slot, nh, chunk);
 }
 
 template <typename T>
