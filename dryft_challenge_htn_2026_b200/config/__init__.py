@@ -4,9 +4,10 @@ from .specs import (AttentionSpec, DenseMLPSpec, GatedLinearAttentionSpec, Gated
                     MaskedAttentionSpec, ModelSpec, OnePlusRMSNormSpec, ParallelMixerSpec, PostNormLayerSpec, RMSNormSpec,
                     RotaryHalfSpec, RotaryPairsSpec, RotaryPartSpec, RoutedMLPSpec, SandwichLayerSpec, ScalarRMSNormSpec, ScheduleEntry,
                     SinusoidSpec, UnitRMSNormSpec, LatentAttentionSpec, DiffAttentionSpec, GroupRMSNormSpec,
-                    LowerBoundRecurrenceSpec, StateSpaceSpec, BigramSpec, GatedDeltaSpec, LayerNormSpec, OutputNormLayerSpec)
+                    LowerBoundRecurrenceSpec, StateSpaceSpec, BigramSpec, GatedDeltaSpec, LayerNormSpec, MatrixMemorySpec, OutputNormLayerSpec)
 from .base import ConfigError, ModelConfig
 from .fukatar import FukatarConfig
+from .mozutar import MozutarConfig
 from .nevotar import NevotarConfig
 from .nilivik import NilivikConfig
 from .pibulix import PibulixConfig
@@ -18,5 +19,5 @@ __all__ = ["AttentionSpec", "DenseMLPSpec", "GatedMLPSpec", "LayerSpec", "Linear
            "SinusoidSpec", "ConfigError", "ModelConfig", "NilivikConfig", "Qwen3Config", "PibulixConfig",
            "GatedLinearAttentionSpec", "OnePlusRMSNormSpec", "PostNormLayerSpec", "RotaryPartSpec", "RoutedMLPSpec", "VenidraConfig", "LatentAttentionSpec", "RotaryPairsSpec",
            "SandwichLayerSpec", "UnitRMSNormSpec", "NevotarConfig", "DiffAttentionSpec", "GroupRMSNormSpec",
-           "LowerBoundRecurrenceSpec", "StateSpaceSpec", "FukatarConfig", "BigramSpec", "GatedDeltaSpec", "LayerNormSpec",
+           "LowerBoundRecurrenceSpec", "StateSpaceSpec", "FukatarConfig", "MozutarConfig", "MatrixMemorySpec", "BigramSpec", "GatedDeltaSpec", "LayerNormSpec",
            "OutputNormLayerSpec"]

@@ -27,6 +27,8 @@ def linear(x, w, mode=STORE, allow_partial=False, act=(0.0, 0.0)):
         out = torch.empty((M, N), dtype=torch.float32, device=x.device)
         api.sgemm(x, w, out, mode, act)
         return out
+    if x.data_ptr() % 16:        # a single row cut out of a wider one is dense where it lies: the products read 16 bytes at a time
+        x = x.clone()
     if K % 8:
         # an inner size the tensor-core kernels do not take (their rows sit on 16-byte boundaries): the library's
         # product, and the activation as a row kernel behind it

@@ -23,7 +23,7 @@ from dryft_challenge_htn_2026_b200.csrc import api
 from dryft_challenge_htn_2026_b200.engine import DecodeLoop, Runner, load_model
 from dryft_challenge_htn_2026_b200.parts import Runtime, build_part
 from helpers import ROOT, random_tokens
-from part_helpers import DEV, bound_part, close, dev, rnd, run_cut, tol, whole
+from part_helpers import DEV, Errors, bound_part, close, dev, rnd, run_cut, tol, whole
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
@@ -452,27 +452,6 @@ def test_two_mixers_side_by_side_with_normed_outputs(dtype, left, right):
 
 
 # ------------------------------------------------------------------------------------ whole models
-class Errors:
-    """float32 must hold everywhere. In bfloat16 a position now and then lies far off by rounding alone: a head's output that
-    nearly vanishes is blown up by the norm over its own root mean square, and the rounding in it too (the plain
-    implementation with every activation rounded to bfloat16 leaves the same positions off). One in twenty may be, none by
-    more than eight times the tolerance; a fault in a kernel puts nearly all of them off."""
-
-    def __init__(self, dtype):
-        self.dtype, self.n, self.bad = dtype, 0, []
-
-    def add(self, got, ref, what, bound_of=None):
-        err, bound = float((got.double().cpu() - ref).abs().max()), tol(self.dtype, ref if bound_of is None else bound_of)
-        self.n += 1
-        if err > bound:
-            self.bad.append((what, err, bound))
-
-    def verdict(self):
-        exact = self.dtype in (torch.float32, "float32")
-        assert len(self.bad) <= (0 if exact else 1 + self.n // 20), f"{len(self.bad)} of {self.n} positions off: {self.bad[:5]}"
-        assert all(err <= 8 * bound for _, err, bound in self.bad), self.bad
-
-
 def plain_logits(folder, tokens):
     cfg, t = plain.read_model(folder)
     return plain.forward(tokens, t, cfg)
