@@ -95,6 +95,61 @@ moe_scores_kernel(const T* x, int W, const float* __restrict__ wr, const float* 
     }
 }
 
+// The same for up to 8 tokens: a block per router row, its warps share the row's elements out (with eight rows a block a
+// single-token step had a handful of blocks, each a chain of a warp's loads: 23 us for 32 rows of 2,560).
+template <typename T>
+__global__ void __launch_bounds__(32 * ROUTE_WARPS)
+moe_scores_few_kernel(const T* x, int W, const float* __restrict__ wr, const float* __restrict__ wsg, int E, float* scores,
+                      float* sgate, int n_tok, int by_logit) {
+    __shared__ float part[ROUTE_WARPS][ROUTE_TOKENS];
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, e = blockIdx.x;
+    const float* row = e < E ? wr + (size_t)e * W : wsg;
+    pdl_wait();
+    pdl_launch_dependents();
+    float acc[ROUTE_TOKENS];
+#pragma unroll
+    for (int tt = 0; tt < ROUTE_TOKENS; tt++) acc[tt] = 0.f;
+    if (W % 4 == 0) {
+        for (int k = (w * 32 + lane) * 4; k < W; k += 128 * ROUTE_WARPS) {
+            const float4 r = __ldg(reinterpret_cast<const float4*>(row + k));
+#pragma unroll
+            for (int tt = 0; tt < ROUTE_TOKENS; tt++) {
+                if (tt >= n_tok) continue;
+                float xv[4];
+                if (sizeof(T) == 2) {
+                    const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(x) + (size_t)tt * W + k);
+                    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+                    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+                    xv[0] = a.x, xv[1] = a.y, xv[2] = b.x, xv[3] = b.y;
+                } else {
+                    const float4 a = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(x) + (size_t)tt * W + k);
+                    xv[0] = a.x, xv[1] = a.y, xv[2] = a.z, xv[3] = a.w;
+                }
+                acc[tt] = fmaf(r.x, xv[0], fmaf(r.y, xv[1], fmaf(r.z, xv[2], fmaf(r.w, xv[3], acc[tt]))));
+            }
+        }
+    } else {
+        for (int k = w * 32 + lane; k < W; k += 32 * ROUTE_WARPS)
+#pragma unroll
+            for (int tt = 0; tt < ROUTE_TOKENS; tt++)
+                if (tt < n_tok) acc[tt] = fmaf(row[k], to_f(x[(size_t)tt * W + k]), acc[tt]);
+    }
+#pragma unroll
+    for (int tt = 0; tt < ROUTE_TOKENS; tt++) {
+        const float z = warp_sum(acc[tt]);
+        if (lane == 0) part[w][tt] = z;
+    }
+    __syncthreads();
+    const int tt = threadIdx.x;
+    if (tt >= n_tok) return;
+    float z = 0.f;
+#pragma unroll
+    for (int i = 0; i < ROUTE_WARPS; i++) z += part[i][tt];
+    const float sg = 1.f / (1.f + expf(-z));
+    if (e < E) scores[(size_t)tt * E + e] = by_logit ? z : sg;
+    else sgate[tt] = sg;
+}
+
 // Choice: a warp a token, from the token's scores.
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
 moe_choose_kernel(const float* scores, const float* __restrict__ corr, int E, int top, int groups, int keep, float scale,
@@ -281,42 +336,64 @@ moe_down_rows_kernel(const T* mid, const T* __restrict__ wd, int E, const int* i
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
-    for (int i = threadIdx.x; i < top * ff; i += blockDim.x)
-        if (idx[(size_t)t * top + i / ff] < E)
-            ms[i] = to_f(mid[(size_t)t * top * ff + i]) * (wt != nullptr ? wt[(size_t)t * top + i / ff] : 1.f);
+    for (int j = 0; j < top; j++) {
+        const size_t pair = (size_t)t * top + j;
+        if (idx[pair] >= E) continue;
+        const float f = wt != nullptr ? wt[pair] : 1.f;
+        for (int k = threadIdx.x; k < ff; k += blockDim.x) ms[j * ff + k] = to_f(mid[pair * ff + k]) * f;
+    }
     __syncthreads();
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
     const int c_end = min(W, (int)(blockIdx.y + 1) * rows_per_block);
-    constexpr int N = Vec<T>::N;
-    for (int c = blockIdx.y * rows_per_block + w; c < c_end; c += 4) {
-        float acc = 0.f;
+    constexpr int N = Vec<T>::N, R = 2;          // R columns of the output a warp at a time: twice the requests in flight
+    for (int c0 = blockIdx.y * rows_per_block + w; c0 < c_end; c0 += 4 * R) {
+        float acc[R];
+        int c[R];
+#pragma unroll
+        for (int r = 0; r < R; r++) acc[r] = 0.f, c[r] = min(c0 + 4 * r, c_end - 1);     // past the end: the last column again, not stored
         for (int j = 0; j < top; j++) {
-            if (idx[(size_t)t * top + j] >= E) {
-                const float* w = wt != nullptr ? wt : in_wt;
-                if (lane == 0) acc = fmaf(w != nullptr ? w[(size_t)t * top + j] : 1.f, to_f(x[(size_t)t * W + c]), acc);
+            const size_t pair = (size_t)t * top + j;
+            const int e = idx[pair];
+            if (e >= E) {
+                const float* f = wt != nullptr ? wt : in_wt;
+                if (lane == 0)
+#pragma unroll
+                    for (int r = 0; r < R; r++) acc[r] = fmaf(f != nullptr ? f[pair] : 1.f, to_f(x[(size_t)t * W + c[r]]), acc[r]);
                 continue;
             }
-            const T* row = wd + ((size_t)idx[(size_t)t * top + j] * W + c) * ff;
-            float a = 0.f;
+            const T* rows[R];
+            float a[R];
+#pragma unroll
+            for (int r = 0; r < R; r++) rows[r] = wd + ((size_t)e * W + c[r]) * ff, a[r] = 0.f;
             if (VEC) {
 #pragma unroll 4
                 for (int k = lane * N; k < ff; k += 32 * N) {
-                    float rv[N], mv[N];
-                    Vec<T>::load(row + k, rv);
+                    float mv[N];
 #pragma unroll
                     for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(mv + i) = *reinterpret_cast<const float4*>(ms + j * ff + k + i);
 #pragma unroll
-                    for (int i = 0; i < N; i++) a = fmaf(rv[i], mv[i], a);
+                    for (int r = 0; r < R; r++) {
+                        float rv[N];
+                        Vec<T>::load(rows[r] + k, rv);
+#pragma unroll
+                        for (int i = 0; i < N; i++) a[r] = fmaf(rv[i], mv[i], a[r]);
+                    }
                 }
             } else {
-                for (int k = lane; k < ff; k += 32) a = fmaf(to_f(row[k]), ms[j * ff + k], a);
+                for (int k = lane; k < ff; k += 32)
+#pragma unroll
+                    for (int r = 0; r < R; r++) a[r] = fmaf(to_f(rows[r][k]), ms[j * ff + k], a[r]);
             }
-            acc += a;
+#pragma unroll
+            for (int r = 0; r < R; r++) acc[r] += a[r];
         }
-        acc = warp_sum(acc);
-        if (lane == 0) {
-            if (shared != nullptr) acc = fmaf(sgate ? sgate[t] : 1.f, to_f(shared[(size_t)t * W + c]), acc);
-            out[(size_t)t * W + c] = from_f<T>(acc);
+#pragma unroll
+        for (int r = 0; r < R; r++) {
+            float y = warp_sum(acc[r]);
+            if (lane == 0 && c0 + 4 * r < c_end) {
+                if (shared != nullptr) y = fmaf(sgate ? sgate[t] : 1.f, to_f(shared[(size_t)t * W + c[r]]), y);
+                out[(size_t)t * W + c[r]] = from_f<T>(y);
+            }
         }
     }
 }
@@ -324,6 +401,9 @@ moe_down_rows_kernel(const T* mid, const T* __restrict__ wd, int E, const int* i
 template <typename T>
 static int launch_scores(const void* x, int W, const float* wr, const float* wsg, int E, float* scores, float* sgate, int n_tok,
                          int by_logit, cudaStream_t st) {
+    if (n_tok <= ROUTE_TOKENS)
+        return dk_launch(moe_scores_few_kernel<T>, dim3(E + (wsg != nullptr ? 1 : 0)), dim3(32 * ROUTE_WARPS), 0, st, (const T*)x, W, wr, wsg, E,
+                         scores, sgate, n_tok, by_logit);
     const size_t smem = sizeof(T) * (size_t)ROUTE_TOKENS * W;
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_scores_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
